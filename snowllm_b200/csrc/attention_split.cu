@@ -11,6 +11,7 @@
 //     more term exp(sink) in the softmax's sum, without a key or a value);
 //   * `keep` > 0: beside its window a query reaches the positions below `keep` (the sequence's first tokens);
 //   * bias_len < 0: `bias` holds one slope per query head and slope * (i - j) is taken off the scaled score;
+//   * `softcap` c > 0: the scaled score becomes c tanh(score / c), ahead of bias, slope and mask;
 //   * `gate`: a logit per (row, query head); the head's output is multiplied by its sigmoid;
 //   * scores, softmax weights and the products with the values in float whatever the cache dtype (the
 //     weights are never rounded to 16 bits), output in float or in the compute dtype.
@@ -58,6 +59,16 @@ template <int N> __device__ __forceinline__ void sa_cp_async_wait() {
 }
 
 // ---------------------------------------------------------------------------------------------
+// Values that go over, row by row, into another layer's values of the same tokens: (1 - lambda) v + lambda v_first.
+// first: that layer's value columns [nkv, dv] in its projection's rows (row pitch ld), bias the biases of those
+// columns (may be null); first null: nothing is mixed.
+struct ValueMix {
+  const void* first;
+  long long ld;
+  const float* bias;
+  float lambda;
+};
+
 // One warp per (row, head) of q, k and v.  proj: the fused projection's output, row pitch ld, with q at
 // column q_off ([nq, dk]), k at k_off ([nkh, dk], nkh = kv heads * maps) and v at v_off ([nkv, dv]).
 template <typename T>
@@ -68,7 +79,7 @@ __global__ void split_prepare_kernel(const T* __restrict__ proj, long long ld, i
                                      const int* __restrict__ positions, const int* __restrict__ row_seg,
                                      const int* __restrict__ block_table, int max_pages, int page_size,
                                      T* __restrict__ kpool, T* __restrict__ vpool, T* __restrict__ q_out,
-                                     int nq, int nkh, int nkv, int dk, int dv, int write_kv) {
+                                     int nq, int nkh, int nkv, int dk, int dv, int write_kv, ValueMix mix) {
   pdl_begin();
   extern __shared__ float sp_sh[];                     // [warps][dk]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -84,7 +95,14 @@ __global__ void split_prepare_kernel(const T* __restrict__ proj, long long ld, i
     const int h = unit - nq - nkh;
     const T* src = row + v_off + (size_t)h * dv;
     T* dst = vpool + (((size_t)page * nkv + h) * page_size + pos % page_size) * dv;
-    if (proj_bias) {
+    if (mix.first) {
+      for (int d = lane; d < dv; d += 32) {
+        const int c = h * dv + d;
+        const float own = to_f<T>(src[d]) + (proj_bias ? proj_bias[v_off + c] : 0.f);
+        const float first = to_f<T>(static_cast<const T*>(mix.first)[(size_t)m * mix.ld + c]) + (mix.bias ? mix.bias[c] : 0.f);
+        dst[d] = from_f<T>(fmaf(mix.lambda, first, (1.f - mix.lambda) * own));
+      }
+    } else if (proj_bias) {
       const float* bs = proj_bias + v_off + (size_t)h * dv;
       for (int d = lane; d < dv; d += 32) dst[d] = from_f<T>(to_f<T>(src[d]) + bs[d]);
     } else {
@@ -165,7 +183,7 @@ split_prepare_vec_kernel(const T* __restrict__ proj, long long ld, int q_off, in
                          const int* __restrict__ positions, const int* __restrict__ row_seg,
                          const int* __restrict__ block_table, int max_pages, int page_size,
                          T* __restrict__ kpool, T* __restrict__ vpool, T* __restrict__ q_out,
-                         int nq, int nkh, int nkv, int dk, int dv, int write_kv) {
+                         int nq, int nkh, int nkv, int dk, int dv, int write_kv, ValueMix mix) {
   pdl_begin();
   constexpr int VEC = SaVec<T>::N;
   __shared__ float red[33];
@@ -273,6 +291,15 @@ split_prepare_vec_kernel(const T* __restrict__ proj, long long ld, int q_off, in
     } else {
       const int vv = v - nqv - nkv_;
       const int hh = vv / vph, lv = vv - hh * vph;
+      if (mix.first) {
+        float f[VEC];
+        SaVec<T>::unpack(*reinterpret_cast<const uint4*>(static_cast<const T*>(mix.first) + (size_t)m * mix.ld + vv * VEC), f);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          const float first = f[e] + (mix.bias ? mix.bias[vv * VEC + e] : 0.f);
+          x[it][e] = fmaf(mix.lambda, first, (1.f - mix.lambda) * x[it][e]);
+        }
+      }
       dst = vpool + (((size_t)page * nkv + hh) * page_size + pos % page_size) * dv + lv * VEC;
     }
 #pragma unroll
@@ -285,11 +312,13 @@ SNK_API int snk_split_prepare(const void* proj, long long ld, int q_off, int k_o
                               const void* k_gamma, int gamma_f32, int has_norm, float eps, const float* inv_freq,
                               int rot_dim, float rot_mult, const int* positions, const int* row_seg,
                               const int* block_table, int max_pages, int page_size, void* kpool, void* vpool,
-                              void* q_out, int M, int nq, int nkh, int nkv, int dk, int dv, int write_kv, int dtype,
-                              cudaStream_t stream) {
+                              void* q_out, int M, int nq, int nkh, int nkv, int dk, int dv, int write_kv,
+                              const void* mix_first, long long mix_ld, const float* mix_bias, float mix_lambda,
+                              int dtype, cudaStream_t stream) {
   if (M <= 0) return 0;
   if (nq <= 0 || dk <= 0 || rot_dim < 0 || rot_dim > dk || (rot_dim & 1)) return SNK_ERR_SIZE;
   if (write_kv && (nkv <= 0 || nkh <= 0 || nkh % nkv || dv <= 0)) return SNK_ERR_SIZE;
+  const ValueMix mix{write_kv ? mix_first : nullptr, mix_ld, mix_bias, mix_lambda};
   {
     // rows of 16-byte vectors whose heads' lanes fit a warp: the vector kernel
     const int vec = dtype == SNK_F32 ? 4 : 8;
@@ -300,7 +329,8 @@ SNK_API int snk_split_prepare(const void* proj, long long ld, int q_off, int k_o
                       (rot_dim / 2) % vec == 0 && q_off % vec == 0 && (!write_kv || (k_off % vec == 0 && v_off % vec == 0)) &&
                       ld % vec == 0 && (uintptr_t)proj % 16 == 0 && (uintptr_t)q_out % 16 == 0 &&
                       (!write_kv || ((uintptr_t)kpool % 16 == 0 && (uintptr_t)vpool % 16 == 0)) && total <= 256 * 8 &&
-                      (rot_dim == 0 || inv_freq != nullptr) && esz * vec == 16;
+                      (rot_dim == 0 || inv_freq != nullptr) && esz * vec == 16 &&
+                      (uintptr_t)mix.first % 16 == 0 && mix.ld % vec == 0;
     if (fits && M <= 2147483647) {
       const int iters = (total + 255) / 256;
       const size_t tab = (size_t)(rot_dim / 2) * sizeof(float2);
@@ -308,7 +338,7 @@ SNK_API int snk_split_prepare(const void* proj, long long ld, int q_off, int k_o
   snk_launch(split_prepare_vec_kernel<T, I_>, dim3(M), dim3(256), tab, stream, static_cast<const T*>(proj), ld,    \
              q_off, k_off, v_off, proj_bias, SmallVec{q_gamma, gamma_f32}, SmallVec{k_gamma, gamma_f32}, has_norm,  \
              eps, inv_freq, rot_dim, rot_mult, positions, row_seg, block_table, max_pages, page_size,            \
-             static_cast<T*>(kpool), static_cast<T*>(vpool), static_cast<T*>(q_out), nq, nkh, nkv, dk, dv, write_kv)
+             static_cast<T*>(kpool), static_cast<T*>(vpool), static_cast<T*>(q_out), nq, nkh, nkv, dk, dv, write_kv, mix)
       SNK_DISPATCH(dtype, {
         if (iters <= 1) SP_VEC(1);
         else if (iters <= 2) SP_VEC(2);
@@ -330,7 +360,7 @@ SNK_API int snk_split_prepare(const void* proj, long long ld, int q_off, int k_o
                                  SmallVec{q_gamma, gamma_f32}, SmallVec{k_gamma, gamma_f32}, has_norm, eps, inv_freq,
                                  rot_dim, rot_mult, positions, row_seg, block_table, max_pages, page_size,
                                  static_cast<T*>(kpool), static_cast<T*>(vpool), static_cast<T*>(q_out), nq, nkh,
-                                 nkv, dk, dv, write_kv));
+                                 nkv, dk, dv, write_kv, mix));
   SNK_LAUNCH_CHECK();
   return 0;
 }
@@ -343,7 +373,7 @@ __global__ void split_attention_kernel(
     const int* __restrict__ block_table, int max_pages, int page_size, const int* __restrict__ positions,
     const int* __restrict__ row_seg, const int* __restrict__ tiles, void* __restrict__ out, int out_f32,
     int nq, int nkv, int maps, int dk, int dv, int window, float scale, const float* __restrict__ bias,
-    int bias_len, const float* __restrict__ head_scale, const float* __restrict__ sink, int keep,
+    int bias_len, const float* __restrict__ head_scale, const float* __restrict__ sink, int keep, float softcap,
     const T* __restrict__ gate, long long gate_ld, int vec_ok, int chunk,
     int num_chunks, float* __restrict__ part_o, float* __restrict__ part_ml) {
   pdl_begin();
@@ -482,6 +512,7 @@ __global__ void split_attention_kernel(
         const T* kr = reinterpret_cast<const T*>(ks + lane * k_stride) + map * dk;
         for (int d = 0; d < dk; ++d) s = fmaf(qw[d], to_f<T>(kr[d]), s);
       }
+      if (softcap > 0.f) s = softcap * tanhf(s / softcap);
       if (bias && valid)
         s = bias_len < 0 ? fmaf(-bias[kvh * hpv + hh], (float)(p - kp), s)
                          : s + bias[(size_t)(kvh * hpv + hh) * bias_len + min(p - kp, bias_len - 1)];
@@ -576,13 +607,17 @@ __device__ __forceinline__ float ex2_approx(float x) {
   return y;
 }
 
+// tanh(z) from 2 log2(e) z: 1 - 2 / (e^(2z) + 1), with the special-function unit's exponential and reciprocal
+// (within 3e-7 of the exact value; -1 and 1 at the ends).
+__device__ __forceinline__ float tanh_of_log2(float x) { return 1.f - __fdividef(2.f, ex2_approx(x) + 1.f); }
+
 template <int DKS, int DVT>
 __global__ void split_attention_mma_kernel(
     const bf16* __restrict__ q, const bf16* __restrict__ kpool, const bf16* __restrict__ vpool,
     const int* __restrict__ block_table, int max_pages, int page_size, const int* __restrict__ positions,
     const int* __restrict__ row_seg, const int* __restrict__ tiles, void* __restrict__ out, int out_f32,
     int nq, int nkv, int maps, int dk, int dv, int window, float scale, const float* __restrict__ bias,
-    int bias_len, const float* __restrict__ head_scale, const float* __restrict__ sink, int keep,
+    int bias_len, const float* __restrict__ head_scale, const float* __restrict__ sink, int keep, float softcap,
     const bf16* __restrict__ gate, long long gate_ld, int chunk, int num_chunks,
     float* __restrict__ part_o, float* __restrict__ part_ml) {
   pdl_begin();
@@ -688,10 +723,14 @@ __global__ void split_attention_mma_kernel(
   };
 
   float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-  float scale2h[2];
+  float scale2h[2], capin[2] = {0.f, 0.f};                 // capin: what turns q . k into 2 log2(e) score / cap
 #pragma unroll
   for (int h2 = 0; h2 < 2; ++h2) {
     scale2h[h2] = head_scale ? scale2 * head_scale[head[h2]] : scale2;
+    if (softcap > 0.f) {
+      capin[h2] = 2.f * scale2h[h2] / softcap;
+      scale2h[h2] = softcap * 1.4426950408889634f;         // of the hyperbolic tangent that takes the score's place
+    }
     if (sink != nullptr && live[h2] && (num_chunks <= 1 || blockIdx.z == 0)) {   // the sink: a term without a key
       mx[h2] = sink[head[h2]] * 1.4426950408889634f;
       l[h2] = 1.f;
@@ -742,6 +781,12 @@ __global__ void split_attention_mma_kernel(
           if (kp * 32 + 16 < dk) mma_bf16_16816(sc[nt], qa[2 * kp + 1], b[2], b[3]);
         }
       }
+    }
+    if (softcap > 0.f) {
+#pragma unroll
+      for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sc[nt][e] = tanh_of_log2(sc[nt][e] * capin[e >> 1]);
     }
     // scale, bias, mask; row maxima over the thread's 8 keys, then over the quad
     // (scores and maxima are kept in units of log 2: the weights are 2^(s - m), one instruction each)
@@ -903,7 +948,7 @@ split_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kpo
                         const int* __restrict__ positions, const int* __restrict__ row_seg,
                         void* __restrict__ out, int out_f32, int nq, int nkv, int maps, int dk, int dv, int window,
                         float scale, const float* __restrict__ bias, int bias_len,
-                        const float* __restrict__ head_scale, const float* __restrict__ sink, int keep,
+                        const float* __restrict__ head_scale, const float* __restrict__ sink, int keep, float softcap,
                         const bf16* __restrict__ gate, long long gate_ld, int num_chunks,
                         float* __restrict__ part_o, float* __restrict__ part_ml) {
   pdl_begin();
@@ -1001,6 +1046,7 @@ split_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kpo
           const int h2 = e >> 1;
           const int kp = t0 + nt * 8 + tq * 2 + (e & 1);
           float sv = sc[nt][e] * (head_scale ? scale2 * head_scale[head[h2]] : scale2);
+          if (softcap > 0.f) sv = softcap * 1.4426950408889634f * tanh_of_log2(sv * (2.f / softcap));
           const bool valid = live[h2] && kp >= lo && kp <= hi;
           if (bias && valid)
             sv = bias_len < 0 ? fmaf(-bias[head[h2]] * (float)(pos - kp), 1.4426950408889634f, sv)
@@ -1160,7 +1206,7 @@ SNK_API int snk_split_attention(const void* q, const void* kpool, const void* vp
                                 int max_pages, int page_size, const int* positions, const int* row_seg,
                                 const int* tiles, int num_tiles, int tile_rows, void* out, int out_f32, int nq,
                                 int nkv, int maps, int dk, int dv, int window, float scale, const float* bias,
-                                int bias_len, const float* head_scale, const float* sink, int keep,
+                                int bias_len, const float* head_scale, const float* sink, int keep, float softcap,
                                 const void* gate, long long gate_ld, int chunk,
                                 int num_chunks, void* scratch, int dtype, cudaStream_t stream) {
   if (num_tiles <= 0) return 0;
@@ -1189,7 +1235,7 @@ SNK_API int snk_split_attention(const void* q, const void* kpool, const void* vp
     snk_launch(split_decode_mma_kernel<DKS_, DVT_>, dim3(grid), dim3(SD_WARPS * 32), smem, stream,           \
                static_cast<const bf16*>(q), static_cast<const bf16*>(kpool), static_cast<const bf16*>(vpool), \
                block_table, max_pages, page_size, positions, row_seg, out, out_f32, nq, nkv, maps, dk, dv,   \
-               window, scale, bias, bias_len, head_scale, sink, keep, static_cast<const bf16*>(gate), gate_ld,   \
+               window, scale, bias, bias_len, head_scale, sink, keep, softcap, static_cast<const bf16*>(gate), gate_ld, \
                num_chunks, part_o, part_ml);                                                                 \
   } while (0)
     if (dk <= 64 && dv <= 64) SD_MMA(4, 8);
@@ -1218,7 +1264,7 @@ SNK_API int snk_split_attention(const void* q, const void* kpool, const void* vp
     snk_launch(split_attention_mma_kernel<DKS_, DVT_>, dim3(grid), dim3(warps * 32), smem, stream,           \
                static_cast<const bf16*>(q), static_cast<const bf16*>(kpool), static_cast<const bf16*>(vpool), \
                block_table, max_pages, page_size, positions, row_seg, tiles, out, out_f32, nq, nkv, maps,    \
-               dk, dv, window, scale, bias, bias_len, head_scale, sink, keep, static_cast<const bf16*>(gate),    \
+               dk, dv, window, scale, bias, bias_len, head_scale, sink, keep, softcap, static_cast<const bf16*>(gate), \
                gate_ld, chunk, num_chunks, part_o, part_ml);                                                 \
   } while (0)
     if (dk <= 64 && dv <= 64) SA_MMA(4, 8);
@@ -1249,7 +1295,7 @@ SNK_API int snk_split_attention(const void* q, const void* kpool, const void* vp
     snk_launch(split_attention_kernel<T, DPL_, UPW_>, dim3(grid), dim3(warps * 32), smem, stream,      \
                static_cast<const T*>(q), static_cast<const T*>(kpool), static_cast<const T*>(vpool),   \
                block_table, max_pages, page_size, positions, row_seg, tiles, out, out_f32, nq, nkv,    \
-               maps, dk, dv, window, scale, bias, bias_len, head_scale, sink, keep,                    \
+               maps, dk, dv, window, scale, bias, bias_len, head_scale, sink, keep, softcap,           \
                static_cast<const T*>(gate), gate_ld, vec_ok, chunk, num_chunks, part_o, part_ml);      \
   } while (0)
 #define SA_LAUNCH_U(DPL_)                  \

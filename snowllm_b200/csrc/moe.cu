@@ -27,6 +27,20 @@
 #define ROUTE_RENORM 1
 #define ROUTE_SOFTMAX 2
 #define ROUTE_PICKED 4
+// Bit 3 (with bit 1): score[] arrives as a correction per expert; the k largest of softmax + correction are picked,
+// and the weights are the softmax without it.
+// Bits 8..17 and 20..29: the experts form that many equal groups of neighbours (0 or 1: no groups), and only experts
+// of the best so many groups can be picked; a group's score is the largest score in it (ties to the lower group).
+#define ROUTE_CORRECTED 8
+#define ROUTE_MAX_GROUPS 128
+__host__ __device__ __forceinline__ int route_groups(int flags) { return (flags >> 8) & 0x3ff; }
+__host__ __device__ __forceinline__ int route_groups_kept(int flags) { return (flags >> 20) & 0x3ff; }
+// Whether the flags fit E experts and k picks.
+static bool route_flags_ok(int flags, int E, int k) {
+  const int count = route_groups(flags), keep = route_groups_kept(flags);
+  if (count <= 1) return true;
+  return count <= ROUTE_MAX_GROUPS && E % count == 0 && keep >= 1 && keep <= count && k <= E / count * keep;
+}
 __device__ __forceinline__ float route_score(float logit, int flags) {
   return (flags & (ROUTE_SOFTMAX | ROUTE_PICKED)) ? logit : 1.f / (1.f + expf(-logit));
 }
@@ -37,6 +51,11 @@ __device__ __forceinline__ void route_put(float logit, const float* __restrict__
     const float z = bias ? logit + bias[e] : logit;
     prob[e] = z;
     score[e] = z;
+    return;
+  }
+  if (flags & ROUTE_CORRECTED) {
+    prob[e] = logit;
+    score[e] = bias[e];
     return;
   }
   const float p = route_score(logit, flags);
@@ -56,7 +75,51 @@ __device__ __forceinline__ void select_topk(float* prob, float* score, int* ids,
     for (int e = lane; e < E; e += 32) den += expf(prob[e] - mx);
     den = warp_sum(den);
     const float inv = 1.f / den;
-    for (int e = lane; e < E; e += 32) prob[e] = expf(prob[e] - mx) * inv;
+    for (int e = lane; e < E; e += 32) {
+      prob[e] = expf(prob[e] - mx) * inv;
+      if (flags & ROUTE_CORRECTED) score[e] += prob[e];
+    }
+    __syncwarp();
+  }
+  const int count = route_groups(flags), groups_kept = route_groups_kept(flags);
+  if (count > 1 && groups_kept < count) {
+    // lane l keeps the scores of groups l, l + 32, ..; a group stays when fewer than `groups_kept` others come before it
+    constexpr int GR = ROUTE_MAX_GROUPS / 32;
+    const int size = E / count;
+    float best[GR];
+#pragma unroll
+    for (int i = 0; i < GR; ++i) best[i] = -INFINITY;
+    for (int g = 0; g < count; ++g) {
+      float mx = -INFINITY;
+      for (int e = lane; e < size; e += 32) mx = fmaxf(mx, score[g * size + e]);
+      mx = warp_max(mx);
+#pragma unroll
+      for (int i = 0; i < GR; ++i)
+        if (g == lane + 32 * i) best[i] = mx;
+    }
+    int before[GR];
+#pragma unroll
+    for (int i = 0; i < GR; ++i) before[i] = 0;
+#pragma unroll
+    for (int j = 0; j < GR; ++j)
+      for (int l = 0; l < 32 && l + 32 * j < count; ++l) {
+        const float other = __shfl_sync(0xffffffffu, best[j], l);
+#pragma unroll
+        for (int i = 0; i < GR; ++i)
+          before[i] += other > best[i] || (other == best[i] && l + 32 * j < lane + 32 * i);
+      }
+    unsigned stays[GR];
+#pragma unroll
+    for (int i = 0; i < GR; ++i)
+      stays[i] = __ballot_sync(0xffffffffu, lane + 32 * i < count && before[i] < groups_kept);
+    for (int e = lane; e < E; e += 32) {
+      const int g = e / size;
+      unsigned mask = stays[0];
+#pragma unroll
+      for (int i = 1; i < GR; ++i)
+        if ((g >> 5) == i) mask = stays[i];
+      if (!((mask >> (g & 31)) & 1u)) score[e] = -INFINITY;
+    }
     __syncwarp();
   }
   float wsum = 0.f;
@@ -222,7 +285,9 @@ __global__ void moe_topk_kernel(const float* __restrict__ logits, const float* _
 SNK_API int snk_moe_topk(const float* logits, const float* bias, int* topk_ids, float* topk_w, int M, int E,
                          int k, int norm_topk, float scaling, int transposed, int planes, cudaStream_t stream) {
   if (M <= 0) return 0;
-  if (E <= 0 || E > ROUTE_MAX_EXPERTS || k <= 0 || k > E || planes < 1 || (planes > 1 && transposed)) return SNK_ERR_SIZE;
+  if (E <= 0 || E > ROUTE_MAX_EXPERTS || k <= 0 || k > E || planes < 1 || (planes > 1 && transposed) ||
+      !route_flags_ok(norm_topk, E, k))
+    return SNK_ERR_SIZE;
   const int warps = 4;
   snk_launch(moe_topk_kernel, dim3((M + warps - 1) / warps), dim3(warps * 32), (size_t)warps * 2 * E * sizeof(float), stream, 
       logits, bias, topk_ids, topk_w, M, E, k, norm_topk, scaling, transposed, planes);
@@ -234,7 +299,7 @@ SNK_API int snk_moe_route(const void* x, const void* wr, int wr_is_f32, const fl
                           int* topk_ids, float* topk_w, int M, int H, int E, int k, int norm_topk,
                           float scaling, int dtype, cudaStream_t stream) {
   if (M <= 0) return 0;
-  if (E <= 0 || E > ROUTE_MAX_EXPERTS || k <= 0 || k > E) return SNK_ERR_SIZE;
+  if (E <= 0 || E > ROUTE_MAX_EXPERTS || k <= 0 || k > E || !route_flags_ok(norm_topk, E, k)) return SNK_ERR_SIZE;
   const size_t smem = (size_t)(2 * E) * sizeof(float);
   SmallVec w{wr, wr_is_f32};
   const size_t xsz = dtype == SNK_F32 ? 4 : 2, wsz = wr_is_f32 ? 4 : 2;
@@ -254,6 +319,8 @@ SNK_API int snk_moe_route(const void* x, const void* wr, int wr_is_f32, const fl
 // ---------------------------------------------------------------------------------------
 // One block sorts all (token, j) pairs by expert.  offsets[E+1]: first sorted row of each
 // expert; pair_pos[p]: sorted row of pair p = m*k + j; sorted_pair[r]: the pair at row r.
+// Experts from `real` on are identity experts (their output is their input): they have no rows of their own in the
+// experts' products, and their pairs' pair_pos is -1.
 // Where a pair lands inside its expert's rows may vary from run to run; no value depends
 // on it, since each row is computed on its own.
 // GLOBAL_IDS: the ids lie in global memory and may have been written by other blocks of this launch, so they
@@ -267,7 +334,7 @@ __device__ __forceinline__ int pair_id(const int* p) {
 template <bool GLOBAL_IDS = false>
 __device__ __forceinline__ void sort_pairs(const int* __restrict__ topk_ids, int* __restrict__ offsets,
                                            int* __restrict__ pair_pos, int* __restrict__ sorted_pair, int pairs,
-                                           int E, int* cnt) {
+                                           int E, int real, int* cnt) {
   int* off = cnt + E;            // cnt: E counts, then E+1 offsets
   for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
@@ -307,7 +374,7 @@ __device__ __forceinline__ void sort_pairs(const int* __restrict__ topk_ids, int
       const int p = threadIdx.x + i * blockDim.x;
       if (p < pairs) {
         const int r = off[ids[i]] + place[i];
-        pair_pos[p] = r;
+        pair_pos[p] = ids[i] < real ? r : -1;
         sorted_pair[r] = p;
       }
     }
@@ -317,17 +384,17 @@ __device__ __forceinline__ void sort_pairs(const int* __restrict__ topk_ids, int
     int e = pair_id<GLOBAL_IDS>(topk_ids + p);
     e = e < 0 ? 0 : (e >= E ? E - 1 : e);
     const int r = off[e] + pair_pos[p];
-    pair_pos[p] = r;
+    pair_pos[p] = e < real ? r : -1;
     sorted_pair[r] = p;
   }
 }
 
 __global__ void moe_sort_kernel(const int* __restrict__ topk_ids, int* __restrict__ offsets,
                                 int* __restrict__ pair_pos, int* __restrict__ sorted_pair, int pairs,
-                                int E) {
+                                int E, int real) {
   pdl_begin();
   extern __shared__ int cnt[];
-  sort_pairs(topk_ids, offsets, pair_pos, sorted_pair, pairs, E, cnt);
+  sort_pairs(topk_ids, offsets, pair_pos, sorted_pair, pairs, E, real, cnt);
 }
 
 // Selection and sort in one block, for the few tokens of a decode step: a warp per token selects from
@@ -336,8 +403,8 @@ __global__ void moe_sort_kernel(const int* __restrict__ topk_ids, int* __restric
 __global__ void moe_topk_sort_kernel(const float* __restrict__ logits, const float* __restrict__ bias,
                                      int* __restrict__ topk_ids, float* __restrict__ topk_w,
                                      int* __restrict__ offsets, int* __restrict__ pair_pos,
-                                     int* __restrict__ sorted_pair, int M, int E, int k, int norm_topk,
-                                     float scaling) {
+                                     int* __restrict__ sorted_pair, int M, int E, int real, int k,
+                                     int norm_topk, float scaling) {
   pdl_begin();
   extern __shared__ float sh[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarp = blockDim.x >> 5;
@@ -356,7 +423,7 @@ __global__ void moe_topk_sort_kernel(const float* __restrict__ logits, const flo
     __syncwarp();
   }
   __syncthreads();
-  sort_pairs(ids_s, offsets, pos_s, sorted_pair, pairs, E, reinterpret_cast<int*>(work));
+  sort_pairs(ids_s, offsets, pos_s, sorted_pair, pairs, E, real, reinterpret_cast<int*>(work));
   __syncthreads();
   for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
     topk_ids[p] = ids_s[p];
@@ -365,11 +432,12 @@ __global__ void moe_topk_sort_kernel(const float* __restrict__ logits, const flo
 }
 
 SNK_API int snk_moe_sort(const int* topk_ids, int* offsets, int* pair_pos, int* sorted_pair,
-                         int pairs, int E, cudaStream_t stream) {
+                         int pairs, int E, int real, cudaStream_t stream) {
   if (pairs <= 0) return 0;
-  if (E <= 0 || E > 4096) return SNK_ERR_SIZE;
+  if (E <= 0 || E > 4096 || real < 0 || real > E) return SNK_ERR_SIZE;
   const size_t smem = (size_t)(2 * E + 1) * sizeof(int);
-  snk_launch(moe_sort_kernel, dim3(1), dim3(1024), smem, stream, topk_ids, offsets, pair_pos, sorted_pair, pairs, E);
+  snk_launch(moe_sort_kernel, dim3(1), dim3(1024), smem, stream, topk_ids, offsets, pair_pos, sorted_pair, pairs, E,
+             real);
   SNK_LAUNCH_CHECK();
   return 0;
 }
@@ -379,10 +447,12 @@ SNK_API int snk_moe_sort(const int* topk_ids, int* offsets, int* pair_pos, int* 
 // the caller then takes snk_moe_route and snk_moe_sort.
 SNK_API int snk_moe_route_sort(const void* x, const void* wr, int wr_is_f32, const float* bias, float* logits,
                                int* topk_ids, float* topk_w, int* offsets, int* pair_pos, int* sorted_pair,
-                               int M, int H, int E, int k, int norm_topk, float scaling, int dtype,
+                               int M, int H, int E, int real, int k, int norm_topk, float scaling, int dtype,
                                cudaStream_t stream) {
   if (M <= 0) return 0;
-  if (E <= 0 || E > ROUTE_MAX_EXPERTS || k <= 0 || k > E || M > 1024) return SNK_ERR_SIZE;
+  if (E <= 0 || E > ROUTE_MAX_EXPERTS || k <= 0 || k > E || M > 1024 || real < 0 || real > E ||
+      !route_flags_ok(norm_topk, E, k))
+    return SNK_ERR_SIZE;
   const int warps = M < 32 ? M : 32;
   size_t smem = (size_t)warps * 2 * E * sizeof(float);
   const size_t sort_smem = (size_t)(2 * E + 1) * sizeof(int);
@@ -398,7 +468,7 @@ SNK_API int snk_moe_route_sort(const void* x, const void* wr, int wr_is_f32, con
                                  static_cast<const T*>(x), w, logits, H, E, vec));
   SNK_LAUNCH_CHECK();
   snk_launch(moe_topk_sort_kernel, dim3(1), dim3(warps * 32), smem, stream, logits, bias, topk_ids, topk_w,
-             offsets, pair_pos, sorted_pair, M, E, k, norm_topk, scaling);
+             offsets, pair_pos, sorted_pair, M, E, real, k, norm_topk, scaling);
   SNK_LAUNCH_CHECK();
   return 0;
 }
@@ -554,7 +624,7 @@ norm_route_sort_kernel(float* __restrict__ residual, const float* __restrict__ d
   __syncthreads();
   if (!is_last) return;
   __threadfence();                                       // the other rows' picks after their tickets
-  sort_pairs<true>(topk_ids, offsets, pair_pos, sorted_pair, M * k, E, reinterpret_cast<int*>(xs));
+  sort_pairs<true>(topk_ids, offsets, pair_pos, sorted_pair, M * k, E, E, reinterpret_cast<int*>(xs));
   if (threadIdx.x == 0) *ticket = 0u;                    // ready for the next launch
 }
 
@@ -598,24 +668,30 @@ SNK_API int snk_norm_route_sort(float* residual, const float* delta, const void*
 }
 
 // ---------------------------------------------------------------------------------------
-// out[m,:] = sum_j w[m,j] * y[pair_pos[m*k+j], :]   (float in, float out)
+// out[m,:] = sum_j w[m,j] * y[pair_pos[m*k+j], :]   (float in, float out); a pair without a row (place -1, an identity
+// expert) stands for the experts' input row x[m, :].
+template <typename T>
 __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ pair_pos,
-                                   const float* __restrict__ topk_w, float* __restrict__ out, int H,
-                                   int k) {
+                                   const float* __restrict__ topk_w, const T* __restrict__ x,
+                                   float* __restrict__ out, int H, int k) {
   pdl_begin();
   const int m = blockIdx.x;
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     float acc = 0.f;
-    for (int j = 0; j < k; ++j)
-      acc = fmaf(topk_w[(size_t)m * k + j], y[(size_t)pair_pos[(size_t)m * k + j] * H + i], acc);
+    for (int j = 0; j < k; ++j) {
+      const int at = pair_pos[(size_t)m * k + j];
+      const float v = at >= 0 ? y[(size_t)at * H + i] : (x ? to_f<T>(x[(size_t)m * H + i]) : 0.f);
+      acc = fmaf(topk_w[(size_t)m * k + j], v, acc);
+    }
     out[(size_t)m * H + i] = acc;
   }
 }
 
-SNK_API int snk_moe_combine(const float* y, const int* pair_pos, const float* topk_w, float* out,
-                            int M, int H, int k, cudaStream_t stream) {
+SNK_API int snk_moe_combine(const float* y, const int* pair_pos, const float* topk_w, const void* x, float* out,
+                            int M, int H, int k, int dtype, cudaStream_t stream) {
   if (M <= 0) return 0;
-  snk_launch(moe_combine_kernel, dim3(M), dim3(H >= 1024 ? 256 : 128), 0, stream, y, pair_pos, topk_w, out, H, k);
+  SNK_DISPATCH(dtype, snk_launch(moe_combine_kernel<T>, dim3(M), dim3(H >= 1024 ? 256 : 128), 0, stream, y, pair_pos,
+                                 topk_w, static_cast<const T*>(x), out, H, k));
   SNK_LAUNCH_CHECK();
   return 0;
 }

@@ -295,11 +295,18 @@ SNK_API int snk_short_conv(const void* bcx, const void* w, int w_is_f32, void* s
 // history holds the same values that a longer step would read from its own rows: a sequence gives the
 // same bits however it is cut.  Launches as above: one that only reads the state and one that rewrites
 // it; steps of one token per segment do both in one.
+__device__ __forceinline__ float conv_silu(float z) { return z / (1.f + expf(-z)); }
+// The taps' sum with the channel's bias (where there is one) and the activation.
+__device__ __forceinline__ float conv_end(float acc, const SmallVec& cb, int c, int silu) {
+  const float z = acc + (cb.p ? cb[c] : 0.f);
+  return silu ? conv_silu(z) : z;
+}
+
 template <typename T>
 __global__ void causal_conv_kernel(const T* __restrict__ u, long long ld, SmallVec w, const T* __restrict__ state,
                                    const int* __restrict__ cu_seqlens, const int* __restrict__ seg_start,
                                    const int* __restrict__ seg_slot, const int* __restrict__ row_seg,
-                                   T* __restrict__ out, long long out_ld, int C, int L) {
+                                   T* __restrict__ out, long long out_ld, int C, int L, SmallVec cb, int silu) {
   pdl_begin();
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   if (c >= C) return;
@@ -318,7 +325,7 @@ __global__ void causal_conv_kernel(const T* __restrict__ u, long long ld, SmallV
     else v = has_state ? to_f<T>(st[(size_t)(s + L - 1) * C + c]) : 0.f;
     acc = fmaf(w[(size_t)c * L + j], v, acc);
   }
-  out[(size_t)m * out_ld + c] = from_f<T>(acc);
+  out[(size_t)m * out_ld + c] = from_f<T>(conv_end(acc, cb, c, silu));
 }
 
 template <typename T>
@@ -351,7 +358,8 @@ __global__ void causal_conv_state_kernel(const T* __restrict__ u, long long ld, 
 template <typename T>
 __global__ void causal_conv_decode_kernel(const T* __restrict__ u, long long ld, SmallVec w, T* __restrict__ state,
                                           const int* __restrict__ seg_start, const int* __restrict__ seg_slot,
-                                          T* __restrict__ out, long long out_ld, int C, int L) {
+                                          T* __restrict__ out, long long out_ld, int C, int L, SmallVec cb,
+                                          int silu) {
   pdl_begin();
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   if (c >= C) return;
@@ -368,7 +376,7 @@ __global__ void causal_conv_decode_kernel(const T* __restrict__ u, long long ld,
   for (int j = 0; j < CONV_MAX_L; ++j)
     if (j < L - 1) acc = fmaf(w[(size_t)c * L + j], to_f<T>(hist[j]), acc);
   acc = fmaf(w[(size_t)c * L + L - 1], to_f<T>(cur), acc);
-  out[(size_t)seg * out_ld + c] = from_f<T>(acc);
+  out[(size_t)seg * out_ld + c] = from_f<T>(conv_end(acc, cb, c, silu));
 #pragma unroll
   for (int j = 0; j < CONV_MAX_L; ++j)
     if (j < L - 1) st[(size_t)j * C + c] = j + 1 < L - 1 ? hist[j + 1] : cur;
@@ -382,7 +390,7 @@ __global__ void __launch_bounds__(128)
 causal_conv_strip_kernel(const T* __restrict__ u, long long ld, SmallVec w, const T* __restrict__ state,
                          const int* __restrict__ cu_seqlens, const int* __restrict__ seg_start,
                          const int* __restrict__ seg_slot, const int* __restrict__ row_seg,
-                         T* __restrict__ out, long long out_ld, int M, int C) {
+                         T* __restrict__ out, long long out_ld, int M, int C, SmallVec cb, int silu) {
   pdl_begin();
   constexpr int VEC = ConvVec<T>::N;
   using Raw = typename ConvVec<T>::Raw;
@@ -408,6 +416,9 @@ causal_conv_strip_kernel(const T* __restrict__ u, long long ld, SmallVec w, cons
   for (int j = 0; j < L; ++j)
 #pragma unroll
     for (int e = 0; e < VEC; ++e) taps[j][e] = w[(size_t)(c0 + e) * L + j];
+  float bias[VEC];
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) bias[e] = cb.p ? cb[c0 + e] : 0.f;
   float hist[L - 1][VEC];                            // hist[0] is the oldest of the L-1 values before the row
   int seg = -1;
 #pragma unroll
@@ -441,7 +452,7 @@ causal_conv_strip_kernel(const T* __restrict__ u, long long ld, SmallVec w, cons
 #pragma unroll
         for (int i = 0; i < L - 1; ++i) acc = fmaf(taps[i][e], hist[i][e], acc);
         acc = fmaf(taps[L - 1][e], x[e], acc);
-        y[e] = acc;
+        y[e] = silu ? conv_silu(acc + bias[e]) : acc + bias[e];
 #pragma unroll
         for (int i = 0; i < L - 2; ++i) hist[i][e] = hist[i + 1][e];
         if (L > 1) hist[L - 2 < 0 ? 0 : L - 2][e] = x[e];
@@ -451,19 +462,20 @@ causal_conv_strip_kernel(const T* __restrict__ u, long long ld, SmallVec w, cons
   }
 }
 
+// bias (may be null, float when the taps are): added to the taps' sum; silu: the activation z * sigmoid(z) on top.
 SNK_API int snk_causal_conv(const void* u, long long ld, const void* w, int w_is_f32, void* state,
                             const int* cu_seqlens, const int* seg_start, const int* seg_slot, const int* row_seg,
-                            void* out, long long out_ld, int M, int B, int C, int L, int dtype,
-                            cudaStream_t stream) {
+                            void* out, long long out_ld, int M, int B, int C, int L, const void* bias, int silu,
+                            int dtype, cudaStream_t stream) {
   if (M <= 0 || B <= 0 || C <= 0) return 0;
   if (L < 1 || L > CONV_MAX_L || M > 65535 * 64 || B > 65535) return SNK_ERR_SIZE;
   const int threads = 128;
-  SmallVec wv{w, w_is_f32};
+  SmallVec wv{w, w_is_f32}, cb{bias, w_is_f32};
   if (M == B && L > 1) {                             // one token per segment
     dim3 dgrid((C + threads - 1) / threads, B);
     SNK_DISPATCH(dtype, snk_launch(causal_conv_decode_kernel<T>, dim3(dgrid), dim3(threads), 0, stream,
                                    static_cast<const T*>(u), ld, wv, static_cast<T*>(state), seg_start, seg_slot,
-                                   static_cast<T*>(out), out_ld, C, L));
+                                   static_cast<T*>(out), out_ld, C, L, cb, silu));
     SNK_LAUNCH_CHECK();
     return 0;
   }
@@ -477,7 +489,7 @@ SNK_API int snk_causal_conv(const void* u, long long ld, const void* w, int w_is
 #define CAUSAL_STRIP_LAUNCH(L_)                                                                          \
     snk_launch(causal_conv_strip_kernel<T, L_>, dim3(sgrid), dim3(threads), 0, stream,                   \
                static_cast<const T*>(u), ld, wv, static_cast<const T*>(state), cu_seqlens, seg_start,    \
-               seg_slot, row_seg, static_cast<T*>(out), out_ld, M, C)
+               seg_slot, row_seg, static_cast<T*>(out), out_ld, M, C, cb, silu)
     SNK_DISPATCH(dtype, {
       if (L == 2) CAUSAL_STRIP_LAUNCH(2);
       else if (L == 3) CAUSAL_STRIP_LAUNCH(3);
@@ -489,7 +501,7 @@ SNK_API int snk_causal_conv(const void* u, long long ld, const void* w, int w_is
     dim3 grid((C + threads - 1) / threads, M);
     SNK_DISPATCH(dtype, snk_launch(causal_conv_kernel<T>, dim3(grid), dim3(threads), 0, stream,
                                    static_cast<const T*>(u), ld, wv, static_cast<const T*>(state), cu_seqlens,
-                                   seg_start, seg_slot, row_seg, static_cast<T*>(out), out_ld, C, L));
+                                   seg_start, seg_slot, row_seg, static_cast<T*>(out), out_ld, C, L, cb, silu));
   }
   SNK_LAUNCH_CHECK();
   if (L > 1) {

@@ -64,7 +64,7 @@ class Model:
             yield part
             for inner in getattr(part, "parts", tuple)():
                 yield from walk(inner)
-        yield self.embedding
+        yield from walk(self.embedding)
         for b in self.blocks:
             for p in b.parts():
                 yield from walk(p)
@@ -74,7 +74,7 @@ class Model:
     def libraries(self) -> list[str]:
         """csrc libraries this model's parts launch from (what a first call has to compile)."""
         seen: dict[str, None] = {}
-        for p in self.parts():
+        for p in (*self.parts(), *self.blocks):
             for lib in getattr(p, "libraries", ()):
                 seen[lib] = None
         return list(seen)

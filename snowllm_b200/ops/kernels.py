@@ -33,7 +33,7 @@ _SIGNATURES = {
     },
     "short_conv": {
         "snk_short_conv": [P, P, I, P, P, P, P, P, P, I, I, I, I, I, P],
-        "snk_causal_conv": [P, LL, P, I, P, P, P, P, P, P, LL, I, I, I, I, I, P],
+        "snk_causal_conv": [P, LL, P, I, P, P, P, P, P, P, LL, I, I, I, I, P, I, I, P],
     },
     "attention": {
         "snk_paged_attention_scratch_bytes": [I, I, I, I],
@@ -81,10 +81,10 @@ _SIGNATURES = {
     "moe": {
         "snk_moe_route": [P, P, I, P, P, P, I, I, I, I, I, F, I, P],
         "snk_moe_topk": [P, P, P, P, I, I, I, I, F, I, I, P],
-        "snk_moe_route_sort": [P, P, I, P, P, P, P, P, P, P, I, I, I, I, I, F, I, P],
-        "snk_moe_sort": [P, P, P, P, I, I, P],
+        "snk_moe_route_sort": [P, P, I, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, P],
+        "snk_moe_sort": [P, P, P, P, I, I, I, P],
         "snk_norm_route_sort": [P, P, P, I, P, I, F, P, P, P, I, P, I, P, P, P, P, P, P, I, I, I, I, F, I, P, P],
-        "snk_moe_combine": [P, P, P, P, I, I, I, P],
+        "snk_moe_combine": [P, P, P, P, P, I, I, I, I, P],
         "snk_moe_scaled_rows": [P, P, P, P, P, I, I, I, I, P],
         "snk_row_dot": [P, P, I, P, I, I, I, P],
     },
@@ -104,11 +104,12 @@ _SIGNATURES = {
         "snk_heads_to_rows": [P, P, I, I, I, I, P],
     },
     "attention_split": {
-        "snk_split_prepare": [P, LL, I, I, I, P, P, P, I, I, F, P, I, F, P, P, P, I, I, P, P, P, I, I, I, I, I, I, I, I, P],
+        "snk_split_prepare": [P, LL, I, I, I, P, P, P, I, I, F, P, I, F, P, P, P, I, I, P, P, P, I, I, I, I, I, I, I, P, LL, P, F, I,
+                              P],
         "snk_split_attention_tile_rows": [I, I, I, I, I, I, I],
         "snk_split_attention_decode_chunk": [I, I, I, I, I, I],
-        "snk_split_attention": [P, P, P, P, I, I, P, P, P, I, I, P, I, I, I, I, I, I, I, F, P, I, P, P, I, P, LL, I, I, P,
-                                I, P],
+        "snk_split_attention": [P, P, P, P, I, I, P, P, P, I, I, P, I, I, I, I, I, I, I, F, P, I, P, P, I, F, P, LL, I, I,
+                                P, I, P],
     },
     "mlstm": {
         "snk_mlstm": [P, LL, I, I, I, I, I, P, P, I, F, P, P, P, P, P, P, P, I, I, I, I, P],
@@ -119,6 +120,13 @@ _SIGNATURES = {
     "streams": {
         "snk_streams_norm": [P, P, P, P, P, P, P, I, P, P, P, P, I, I, F, P, P, I, I, I, I, I, P],
         "snk_pair_norm_mix": [P, P, P, P, I, F, F, F, P, I, I, P],
+    },
+    "sandwich": {
+        "snk_sandwich_norm": [P, P, P, P, I, P, P, LL, P, P, F, P, LL, I, P, P, F, P, P, I, I, I, P],
+    },
+    "state_space": {
+        "snk_state_space": [P, LL, I, I, I, P, I, LL, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
+        "snk_gate_group_norm": [P, P, LL, P, I, P, I, I, I, F, I, P],
     },
     "sampling": {
         "snk_argmax": [P, P, I, I, P],
@@ -309,14 +317,16 @@ class ExpertSum:
     """A residual delta that is still in pieces: the routed experts' outputs ``y`` [pairs, H] (float), where
     each (token, pick) pair's row lies (``pair_pos`` int32 [M*k]) and the picks' weights (``weights`` float
     [M, k]).  The norm that follows adds sum_j w[m, j] * y[pair_pos[m*k + j]] into the residual itself;
-    ``dense()`` forms the sum for anyone else."""
+    ``dense()`` forms the sum for anyone else.  ``x`` (the experts' input rows [M, H], compute dtype): a pair whose
+    place is -1 (an identity expert) has no row in ``y`` and stands for ``x[m]``; norms that do not know such
+    pairs get the dense sum."""
 
-    def __init__(self, y, pair_pos, weights):
-        self.y, self.pair_pos, self.weights = y, pair_pos, weights
+    def __init__(self, y, pair_pos, weights, x=None):
+        self.y, self.pair_pos, self.weights, self.x = y, pair_pos, weights, x
         self.shape = (weights.shape[0], y.shape[1])
 
     def dense(self) -> torch.Tensor:
-        return moe_combine(self.y, self.pair_pos, self.weights)
+        return moe_combine(self.y, self.pair_pos, self.weights, x=self.x)
 
 
 class DeltaSum:
@@ -333,6 +343,11 @@ class DeltaSum:
         out = self.a.clone() if self.a_gate is None else self.a * torch.sigmoid(self.a_gate[:, :1])
         residual_add(out, self.b.dense() if isinstance(self.b, ExpertSum) else self.b)
         return out
+
+
+def _pieces_with_rows(delta) -> bool:
+    """Whether ``delta`` is an ``ExpertSum`` every pair of which has a row of its own."""
+    return isinstance(delta, ExpertSum) and delta.x is None
 
 
 class ScaledDelta:
@@ -360,10 +375,12 @@ def add_rmsnorm(residual: torch.Tensor, delta, gamma: torch.Tensor, eps: float,
     _chk(residual, "residual", torch.float32)
     moe = gate = None
     dscale = 1.0
+    if isinstance(delta, NormedDelta):
+        return sandwich_norm(residual, delta, gamma, eps, dtype, rows=rows, out=out)
     if isinstance(delta, ScaledDelta):
         delta, dscale = delta.delta, delta.scale
     if isinstance(delta, DeltaSum):
-        if H % 4 == 0 and isinstance(delta.b, ExpertSum) and isinstance(delta.a, torch.Tensor):
+        if H % 4 == 0 and _pieces_with_rows(delta.b) and isinstance(delta.a, torch.Tensor):
             moe, gate, delta = delta.b, delta.a_gate, delta.a
             _chk(moe.y, "expert outputs", torch.float32)
             _chk(moe.pair_pos, "pair positions", torch.int32, (M * moe.weights.shape[1],))
@@ -375,7 +392,7 @@ def add_rmsnorm(residual: torch.Tensor, delta, gamma: torch.Tensor, eps: float,
         else:
             delta = delta.dense()
     if isinstance(delta, ExpertSum):
-        if H % 4 == 0:
+        if H % 4 == 0 and _pieces_with_rows(delta):
             moe, delta = delta, None
             _chk(moe.y, "expert outputs", torch.float32)
             _chk(moe.pair_pos, "pair positions", torch.int32, (M * moe.weights.shape[1],))
@@ -869,11 +886,13 @@ def short_conv(bcx, weight, state, cu_seqlens, seg_start, seg_slot, row_seg, out
 
 # --- matrix products -------------------------------------------------------------------
 
-def causal_conv(u, channels: int, weight, state, cu_seqlens, seg_start, seg_slot, row_seg, out=None):
+def causal_conv(u, channels: int, weight, state, cu_seqlens, seg_start, seg_slot, row_seg, out=None, bias=None,
+                silu: bool = False):
     """Depthwise causal convolution over time on the first ``channels`` columns of ``u`` [M, width]:
     y[t, c] = sum_j weight[c, j] * u~[t - taps + 1 + j, c], where u~ is the request's history (``state``
     [slots, taps-1, channels], the last taps-1 rows of earlier steps; zeros for a fresh request) followed by
-    this step's rows; the state is brought up to date.  Returns y [M, channels]."""
+    this step's rows; the state is brought up to date.  ``bias`` [channels] (in the taps' dtype) is added to the sum;
+    ``silu``: the activation z * sigmoid(z) on top.  Returns y [M, channels]."""
     M, width = u.shape
     dtype = u.dtype
     _chk(u, "conv input", (torch.float32, torch.bfloat16))
@@ -888,9 +907,12 @@ def causal_conv(u, channels: int, weight, state, cu_seqlens, seg_start, seg_slot
     if out is None:
         out = torch.empty(M, C, dtype=dtype, device=u.device)
     _chk(out, "conv output", dtype, (M, C))
+    if bias is not None:
+        _chk(bias, "conv bias", weight.dtype, (C,))
     fused = M == B and L > 1
     check(fn("snk_causal_conv")(_ptr(u), width, _ptr(weight), w32, _ptr(state), _ptr(cu_seqlens), _ptr(seg_start),
-                                _ptr(seg_slot), _ptr(row_seg), _ptr(out), C, M, B, C, L, code_of(dtype), _stream()),
+                                _ptr(seg_slot), _ptr(row_seg), _ptr(out), C, M, B, C, L, _ptr(bias), int(silu), code_of(dtype),
+                                _stream()),
           "causal_conv", launches=1 if fused or L == 1 else 2,
           work=(lambda: (2 * M * C * u.element_size(), 2 * M * C * L)) if fused or L == 1 else
           (lambda: [(2 * M * C * u.element_size(), 2 * M * C * L), (2 * B * (L - 1) * C * u.element_size(), 0)]))
@@ -1099,21 +1121,26 @@ ROUTE_GEMM_MIN_ROWS = 64
 ROUTER_SCORINGS = ("sigmoid", "softmax", "softmax_picked")
 
 
-def _route_flags(norm_topk_prob, scoring: str) -> int:
+def _route_flags(norm_topk_prob, scoring: str, bias=None, groups=(1, 1)) -> int:
     """The routing kernels' ``norm_topk`` argument: bit 0 renormalises the picks' weights by their sum, bit 1
     scores with a softmax over all experts instead of a sigmoid per expert, bit 2 ("softmax_picked") picks by
     the logits themselves (the bias then belongs to the logit) and weights by the softmax over the picked
-    logits alone."""
+    logits alone, bit 3 (a softmax with a ``bias``) adds the bias to the scores that choose.  ``groups`` = (count,
+    keep): only experts of the best ``keep`` of ``count`` equal groups of neighbours can be picked."""
     if scoring not in ROUTER_SCORINGS:
         raise KernelError(f"router scoring {scoring!r} (known: {', '.join(ROUTER_SCORINGS)})")
+    count, keep = groups
+    limits = (int(count) << 8 | int(keep) << 20) if count > 1 else 0
     if scoring == "softmax_picked":
-        return 4
-    return int(bool(norm_topk_prob)) | (2 if scoring == "softmax" else 0)
+        return 4 | limits
+    softmax = (2 | (8 if bias is not None else 0)) if scoring == "softmax" else 0
+    return int(bool(norm_topk_prob)) | softmax | limits
 
 
-def moe_route(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring: str = "sigmoid"):
+def moe_route(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring: str = "sigmoid", groups=(1, 1)):
     """(ids int32 [M, k], weights float [M, k]) of the router, computed in float: a sigmoid per expert, or
-    (``scoring`` "softmax") a softmax over all experts' logits; the k largest scores are picked."""
+    (``scoring`` "softmax") a softmax over all experts' logits; the k largest of score + ``bias`` are picked, among
+    the experts of the best ``groups[1]`` of ``groups[0]`` equal groups; the weights are the scores."""
     M, H = x.shape
     dtype = x.dtype
     _chk(x, "router input", (torch.float32, torch.bfloat16))
@@ -1122,6 +1149,7 @@ def moe_route(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring: str = 
     _chk(router_w, "router weight", shape=(E, H))
     if bias is not None:
         _chk(bias, "expert bias", torch.float32, (E,))
+    flags = _route_flags(norm_topk_prob, scoring, bias, groups)
     ids = torch.empty(M, top_k, dtype=torch.int32, device=x.device)
     wts = torch.empty(M, top_k, dtype=torch.float32, device=x.device)
     if (M > ROUTE_GEMM_MIN_ROWS and router_w.dtype == torch.bfloat16 and gemm_tc_ok(x, router_w)
@@ -1135,7 +1163,7 @@ def moe_route(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring: str = 
                                       _stream()), "gemm_tc_parts",
               work=lambda: (_nbytes(x, router_w) + M * E * 4 * max(planes.value, 1), 2 * M * E * H))
         check(fn("snk_moe_topk")(_ptr(parts), _ptr(bias), _ptr(ids), _ptr(wts), M, E, top_k,
-                                 _route_flags(norm_topk_prob, scoring), float(scaling), 0, planes.value, _stream()), "moe_topk")
+                                 flags, float(scaling), 0, planes.value, _stream()), "moe_topk")
         return ids, wts
     if M > ROUTE_GEMM_MIN_ROWS and router_w.dtype == torch.bfloat16 and gemm_skinny_ok(router_w, x):
         # many rows: the logits are a tensor-core product with float accumulation and float output.  The few
@@ -1143,10 +1171,10 @@ def moe_route(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring: str = 
         # leaves the logits transposed, [E, M].
         logits = gemm_skinny(router_w, x, out_dtype=torch.float32, rows_hint=min(E, 64))
         check(fn("snk_moe_topk")(_ptr(logits), _ptr(bias), _ptr(ids), _ptr(wts), M, E, top_k,
-                                 _route_flags(norm_topk_prob, scoring), float(scaling), 1, 1, _stream()), "moe_topk")
+                                 flags, float(scaling), 1, 1, _stream()), "moe_topk")
         return ids, wts
     check(fn("snk_moe_route")(_ptr(x), _ptr(router_w), w32, _ptr(bias), _ptr(ids), _ptr(wts), M, H, E,
-                              top_k, _route_flags(norm_topk_prob, scoring), float(scaling), code_of(dtype), _stream()),
+                              top_k, flags, float(scaling), code_of(dtype), _stream()),
           "moe_route", work=lambda: (_nbytes(x, router_w, ids, wts), 2 * M * E * H))
     return ids, wts
 
@@ -1154,15 +1182,16 @@ def moe_route(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring: str = 
 ROUTE_FUSED_MAX_ROWS = 32      # up to here: logits spread over the GPU, selection and sort in one block
 
 
-def moe_route_sort(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring: str = "sigmoid"):
+def moe_route_sort(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring: str = "sigmoid", groups=(1, 1),
+                   identity: int = 0):
     """Routing and the sort by expert together: (ids, weights, offsets, pair_pos, sorted_pair) as
     `moe_route` and `moe_sort` give them.  The few rows of a decode step take two launches made for
     them; a row's logits are the same numbers on every path but the tensor-core one."""
     M, H = x.shape
     E = router_w.shape[0]
     if M > ROUTE_FUSED_MAX_ROWS or 8 * E * min(M, 32) + 8 * M * top_k > 48 * 1024:
-        ids, wts = moe_route(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring)
-        return (ids, wts) + moe_sort(ids, E)
+        ids, wts = moe_route(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring, groups)
+        return (ids, wts) + moe_sort(ids, E, identity)
     dtype = x.dtype
     _chk(x, "router input", (torch.float32, torch.bfloat16))
     w32 = _small(router_w, "router weight", dtype)
@@ -1177,8 +1206,9 @@ def moe_route_sort(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring: s
     offsets = ints[3 * pairs:]
     logits, wts = floats[:M * E], floats[M * E:].view(M, top_k)
     check(fn("snk_moe_route_sort")(_ptr(x), _ptr(router_w), w32, _ptr(bias), _ptr(logits), _ptr(ids), _ptr(wts),
-                                   _ptr(offsets), _ptr(pair_pos), _ptr(sorted_pair), M, H, E, top_k,
-                                   _route_flags(norm_topk_prob, scoring), float(scaling), code_of(dtype), _stream()),
+                                   _ptr(offsets), _ptr(pair_pos), _ptr(sorted_pair), M, H, E, E - int(identity), top_k,
+                                   _route_flags(norm_topk_prob, scoring, bias, groups), float(scaling), code_of(dtype),
+                                   _stream()),
           "moe_route_sort", launches=2, work=lambda: (_nbytes(x, router_w, ints, floats), 2 * M * E * H))
     return ids, wts, offsets, pair_pos, sorted_pair
 
@@ -1196,7 +1226,7 @@ def norm_route_sort_ok(residual, delta, gamma, router_w, top_k) -> bool:
     operands (the switch ``FUSE_ROUTER`` is the caller's business)."""
     M, H = residual.shape
     E = router_w.shape[0]
-    plain = delta is None or isinstance(delta, ExpertSum) or (torch.is_tensor(delta) and delta.data_ptr() % 16 == 0)
+    plain = delta is None or _pieces_with_rows(delta) or (torch.is_tensor(delta) and delta.data_ptr() % 16 == 0)
     return (M <= NORM_ROUTE_MAX_ROWS and H % 4 == 0 and H <= 32768 and top_k <= 32 and plain
             and residual.data_ptr() % 16 == 0 and (max(H, 2 * E + 4) + 40 + 2 * E) * 4 <= 200 * 1024)
 
@@ -1257,9 +1287,9 @@ def row_dot(x, w):
     return out
 
 
-def moe_sort(topk_ids, num_experts):
+def moe_sort(topk_ids, num_experts, identity: int = 0):
     """(offsets int32 [E+1], pair_pos int32 [M*k], sorted_pair int32 [M*k]) of the pairs sorted by
-    expert."""
+    expert.  The last ``identity`` experts return their input: their pairs' pair_pos is -1."""
     _chk(topk_ids, "top-k ids", torch.int32)
     pairs = topk_ids.numel()
     dev = topk_ids.device
@@ -1267,12 +1297,12 @@ def moe_sort(topk_ids, num_experts):
     pair_pos = torch.empty(pairs, dtype=torch.int32, device=dev)
     sorted_pair = torch.empty(pairs, dtype=torch.int32, device=dev)
     check(fn("snk_moe_sort")(_ptr(topk_ids), _ptr(offsets), _ptr(pair_pos), _ptr(sorted_pair), pairs,
-                             num_experts, _stream()), "moe_sort")
+                             num_experts, num_experts - int(identity), _stream()), "moe_sort")
     return offsets, pair_pos, sorted_pair
 
 
-def moe_combine(y, pair_pos, topk_w, out=None):
-    """out[m] = sum_j w[m, j] * y[pair_pos[m*k + j]] in float, j in order."""
+def moe_combine(y, pair_pos, topk_w, out=None, x=None):
+    """out[m] = sum_j w[m, j] * y[pair_pos[m*k + j]] in float, j in order; a place of -1 stands for ``x[m]``."""
     M, k = topk_w.shape
     H = y.shape[1]
     _chk(y, "expert outputs", torch.float32, (M * k, H))
@@ -1281,8 +1311,10 @@ def moe_combine(y, pair_pos, topk_w, out=None):
     if out is None:
         out = torch.empty(M, H, dtype=torch.float32, device=y.device)
     _chk(out, "moe output", torch.float32, (M, H))
-    check(fn("snk_moe_combine")(_ptr(y), _ptr(pair_pos), _ptr(topk_w), _ptr(out), M, H, k, _stream()),
-          "moe_combine")
+    if x is not None:
+        _chk(x, "identity rows", (torch.float32, torch.bfloat16), (M, H))
+    check(fn("snk_moe_combine")(_ptr(y), _ptr(pair_pos), _ptr(topk_w), _ptr(x), _ptr(out), M, H, k,
+                                code_of(x.dtype if x is not None else torch.float32), _stream()), "moe_combine")
     return out
 
 
@@ -1462,6 +1494,10 @@ def add_dyt(residual, delta, weight, bias, alpha, dtype, rows=None, out=None):
         da, db = delta.a, delta.b
     elif delta is not None:
         da = delta
+    if isinstance(da, ExpertSum) and da.x is not None:
+        da = da.dense()
+    if isinstance(db, ExpertSum) and db.x is not None:
+        db = db.dense()
     if isinstance(da, ExpertSum):
         da, db = db, da
     if isinstance(db, ExpertSum):
@@ -1634,11 +1670,166 @@ def heads_to_rows(x, out=None):
     return out
 
 
+# --- a norm on both sides of a sublayer ---------------------------------------------------------
+
+class NormedDelta:
+    """A sublayer's update that the norm after it applies in its own kernel (``sandwich_norm``): the raw output ``y``
+    (a float tensor or an ``ExpertSum``; None: no sublayer, the residual is only recorded), ``gate`` = (logits [M,
+    width] in the compute dtype, first column, bias float [H]) whose sigmoid multiplies it element by element, and the
+    output's own RMS norm (``weight`` float [H], ``eps``): x += norm(y * sigmoid(gate)).  ``history`` (float [layers +
+    1, M, H]): the new x is also kept as entry ``index``, and with ``average`` (float [index + 1]) what goes on is
+    sum_j average[j] * history[j]."""
+
+    def __init__(self, y, *, gate=None, weight=None, eps=0.0, history=None, index=0, average=None):
+        self.y, self.gate, self.weight, self.eps = y, gate, weight, float(eps)
+        self.history, self.index, self.average = history, int(index), average
+        self.shape = tuple(y.shape) if y is not None else tuple(history.shape[1:])
+
+    def total(self, residual) -> torch.Tensor:
+        """The residual after the update (for taps and tests, and for norms that do not know this form; not a kernel
+        path).  Nothing is written."""
+        x = residual
+        if self.y is not None:
+            d = self.y.dense() if hasattr(self.y, "dense") else self.y
+            if self.gate is not None:
+                logits, col, bias = self.gate
+                d = d * torch.sigmoid(logits[:, col:col + d.shape[1]].float() + bias)
+            if self.weight is not None:
+                d = d * torch.rsqrt((d * d).mean(-1, keepdim=True) + self.eps) * self.weight
+            x = x + d
+        if self.average is not None:
+            n = self.index
+            x = x * self.average[n] + torch.einsum("j,jmh->mh", self.average[:n], self.history[:n])
+        return x
+
+    def dense(self):
+        raise KernelError("a sublayer's update with a norm of its own does not reduce to a delta that is added: the "
+                          "norm that follows must be one that applies it (rmsnorm)")
+
+
+def sandwich_norm(residual, delta: NormedDelta, weight, eps, dtype, *, rows=None, out=None):
+    """Apply a pending ``NormedDelta`` to the float ``residual`` [M, H] (and to its history) and return the RMS norm
+    of the result times ``weight`` in ``dtype``.  With ``rows`` only those rows come out, and nothing is written
+    back."""
+    M, W = residual.shape
+    _chk(residual, "residual", torch.float32)
+    _chk(weight, "norm weight", torch.float32, (W,))
+    y, moe = delta.y, None
+    if isinstance(y, (ScaledDelta, DeltaSum)):
+        y = y.dense()
+    if isinstance(y, ExpertSum):
+        moe, y = y, y.y
+        _chk(moe.pair_pos, "pair positions", torch.int32, (M * moe.weights.shape[1],))
+        _chk(moe.weights, "top-k weights", torch.float32)
+        _chk(y, "expert outputs", torch.float32)
+        if moe.x is not None:
+            _chk(moe.x, "identity rows", dtype, (M, W))
+    elif y is not None:
+        _chk(y, "sublayer output", torch.float32, (M, W))
+    gate_ptr, gate_ld, gate_bias = c_void_p(0), 0, None
+    if delta.gate is not None and y is not None:
+        logits, col, gate_bias = delta.gate
+        _chk(logits, "output gate", dtype)
+        if logits.dim() != 2 or logits.shape[0] != M or logits.shape[1] < col + W:
+            raise KernelError(f"output gate of shape {tuple(logits.shape)} holds no {W} columns from {col} on")
+        _chk(gate_bias, "output gate bias", torch.float32, (W,))
+        gate_ptr, gate_ld = c_void_p(logits.data_ptr() + col * logits.element_size()), logits.shape[1]
+    if delta.weight is not None:
+        _chk(delta.weight, "output norm weight", torch.float32, (W,))
+    if delta.history is not None:
+        _chk(delta.history, "layer history", torch.float32)
+        if tuple(delta.history.shape[1:]) != (M, W) or not 0 <= delta.index < delta.history.shape[0]:
+            raise KernelError(f"layer history {tuple(delta.history.shape)} has no entry {delta.index} of [{M}, {W}]")
+    if delta.average is not None:
+        if delta.history is None:
+            raise KernelError("a depth average needs the layers' history")
+        _chk(delta.average, "depth average", torch.float32, (delta.index + 1,))
+    R = M if rows is None else rows.numel()
+    if rows is not None:
+        _chk(rows, "norm rows", torch.int32)
+    if out is None:
+        out = torch.empty(R, W, dtype=dtype, device=residual.device)
+    _chk(out, "norm output", dtype, (R, W))
+    k = moe.weights.shape[1] if moe else 0
+    check(fn("snk_sandwich_norm")(
+        _ptr(residual), _ptr(y), _ptr(moe.pair_pos if moe else None), _ptr(moe.weights if moe else None), k,
+        _ptr(moe.x if moe else None), gate_ptr, gate_ld, _ptr(gate_bias),
+        _ptr(delta.weight), delta.eps, _ptr(delta.history), M * W, delta.index, _ptr(delta.average), _ptr(weight),
+        float(eps), _ptr(out), _ptr(rows), R, W, code_of(dtype), _stream()), "sandwich_norm",
+        work=lambda: (R * W * 4 * (1 + (rows is None and (y is not None or delta.average is not None))
+                                   + (max(k, 1) if y is not None else 0)
+                                   + (delta.history is not None and rows is None)
+                                   + (delta.index if delta.average is not None else 0))
+                      + (R * W * out.element_size() if delta.gate is not None else 0) + _nbytes(out), 0))
+    return out
+
+
+# --- state-space recurrence ------------------------------------------------------------------------
+
+def state_space(u, x_off, b_off, c_off, dt, dt_col, dt_bias, rate, skip, cu_seqlens, seg_start, seg_slot, state, groups,
+                max_len, out=None):
+    """S_t = exp(rate[h] step) S_(t-1) + step B_t x_t^T, y_t = S_t^T C_t + skip[h] x_t per (segment, head) over a flat
+    batch, step = softplus(dt + dt_bias[h]).  ``u`` [M, width] (compute dtype) holds x [heads, P] at ``x_off`` and B, C
+    [groups, N] at ``b_off`` and ``c_off``; ``dt`` [M, width'] (float or the compute dtype) one column per head from
+    ``dt_col`` on; ``dt_bias``, ``rate`` (negative), ``skip`` float [heads]; ``state`` float [slots, heads, N, P] is
+    read unless a segment starts at 0, and brought up to date.  ``max_len``: the longest segment.  Returns float [M,
+    heads * P]."""
+    M, width = u.shape
+    dtype = u.dtype
+    _chk(u, "state-space rows", (torch.float32, torch.bfloat16))
+    slots, H, N, Pd = state.shape
+    _chk(state, "state", torch.float32)
+    if width < max(x_off + H * Pd, b_off + groups * N, c_off + groups * N):
+        raise KernelError(f"state-space rows of width {width} are too narrow")
+    _chk(dt, "step projection", (torch.float32, dtype))
+    if dt.dim() != 2 or dt.shape[0] != M or dt.shape[1] < dt_col + H:
+        raise KernelError(f"step projection of shape {tuple(dt.shape)} holds no {H} columns from {dt_col} on")
+    for name, t in (("step bias", dt_bias), ("decay rate", rate), ("skip weight", skip)):
+        _chk(t, name, torch.float32, (H,))
+    B = seg_start.numel()
+    _chk(cu_seqlens, "cu_seqlens", torch.int32, (B + 1,))
+    _chk(seg_start, "seg_start", torch.int32, (B,))
+    _chk(seg_slot, "seg_slot", torch.int32, (B,))
+    if out is None:
+        out = torch.empty(M, H * Pd, dtype=torch.float32, device=u.device)
+    _chk(out, "state-space output", torch.float32, (M, H * Pd))
+    esz = dt.element_size()
+    check(fn("snk_state_space")(_ptr(u), width, int(x_off), int(b_off), int(c_off),
+                                c_void_p(dt.data_ptr() + dt_col * esz), int(dt.dtype == torch.float32), dt.shape[1],
+                                _ptr(dt_bias), _ptr(rate), _ptr(skip), _ptr(cu_seqlens), _ptr(seg_start),
+                                _ptr(seg_slot), _ptr(state), _ptr(out), B, H, int(groups), N, Pd, int(max_len),
+                                code_of(dtype), _stream()), "state_space",
+          work=lambda: ((H * Pd + 2 * groups * N) * M * u.element_size() + M * H * esz + _nbytes(out)
+                        + 2 * B * H * N * Pd * 4, 5 * M * H * N * Pd))
+    return out
+
+
+def gate_group_norm(y, z, z_col, weight, groups, eps, out=None):
+    """v = y * silu(z), each of ``groups`` equal parts of a row over its own sqrt(mean(v^2) + eps), times ``weight``
+    [n], in z's dtype.  ``y`` float [M, n]; ``z`` [M, width] with the gate's n columns from ``z_col`` on."""
+    M, n = y.shape
+    dtype = z.dtype
+    _chk(y, "values to gate", torch.float32)
+    _chk(z, "gate", (torch.float32, torch.bfloat16))
+    if z.dim() != 2 or z.shape[0] != M or z.shape[1] < z_col + n:
+        raise KernelError(f"gate of shape {tuple(z.shape)} holds no {n} columns from {z_col} on")
+    w32 = _small(weight, "norm weight", dtype)
+    _chk(weight, "norm weight", shape=(n,))
+    if out is None:
+        out = torch.empty(M, n, dtype=dtype, device=y.device)
+    _chk(out, "gated values", dtype, (M, n))
+    check(fn("snk_gate_group_norm")(_ptr(y), c_void_p(z.data_ptr() + z_col * z.element_size()), z.shape[1],
+                                    _ptr(weight), w32, _ptr(out), M, n, int(groups), float(eps), code_of(dtype),
+                                    _stream()), "gate_group_norm",
+          work=lambda: (_nbytes(y, out) + M * n * z.element_size(), 0))
+    return out
+
+
 # --- attention over split pools ---------------------------------------------------------------
 
 def split_prepare(proj, q_off, k_off, v_off, q_gamma, k_gamma, eps, inv_freq, rot_dim, rot_mult, positions,
                   row_seg, block_table, page_size, kpool, vpool, nq, nkv, maps, dk, dv, write_kv=True,
-                  proj_bias=None, plain_norm=False, whole_norm=False):
+                  proj_bias=None, plain_norm=False, whole_norm=False, value_mix=None):
     """Rows of a fused projection ``proj`` [M, width] (q at column ``q_off`` as [nq, dk], k at ``k_off`` as
     [nkv*maps, dk], v at ``v_off`` as [nkv, dv]): per-head RMS norm of q and k (if weights are given),
     rotation of the first ``rot_dim`` elements of each head by angle position * inv_freq with cos and sin
@@ -1646,7 +1837,9 @@ def split_prepare(proj, q_off, k_off, v_off, q_gamma, k_gamma, eps, inv_freq, ro
     ([pages, nkv, page_size, maps*dk] and [pages, nkv, page_size, dv]); returns q [M, nq, dk].
     ``proj_bias`` (float [width]): added to the projection's columns first.  ``plain_norm``: q and k over
     their root mean square without a weight.  ``whole_norm``: ONE root mean square over all heads of q (and
-    one over all of k), with weights of the projections' sizes [nq*dk] and [nkv*maps*dk]."""
+    one over all of k), with weights of the projections' sizes [nq*dk] and [nkv*maps*dk].  ``value_mix`` = (rows [M,
+    width'] of another layer's projection, its value columns' offset, its bias over its columns or None, lambda): the
+    values become (1 - lambda) v + lambda v_other."""
     M, width = proj.shape
     dtype = proj.dtype
     _chk(proj, "projection", (torch.float32, torch.bfloat16))
@@ -1675,6 +1868,16 @@ def split_prepare(proj, q_off, k_off, v_off, q_gamma, k_gamma, eps, inv_freq, ro
         if tuple(kpool.shape[1:]) != (nkv, page_size, maps * dk) or tuple(vpool.shape[1:]) != (nkv, page_size, dv):
             raise KernelError(f"pools of shapes {tuple(kpool.shape)} and {tuple(vpool.shape)}, want [pages, {nkv}, "
                               f"{page_size}, {maps * dk}] and [pages, {nkv}, {page_size}, {dv}]")
+    mix_ptr, mix_ld, mix_bias, lam = c_void_p(0), 0, c_void_p(0), 0.0
+    if value_mix is not None and write_kv:
+        first, col, bias, lam = value_mix
+        _chk(first, "values to mix in", dtype)
+        if first.dim() != 2 or first.shape[0] != M or first.shape[1] < col + nkv * dv:
+            raise KernelError(f"values of shape {tuple(first.shape)} hold no {nkv * dv} columns from {col} on")
+        mix_ptr, mix_ld = c_void_p(first.data_ptr() + col * first.element_size()), first.shape[1]
+        if bias is not None:
+            _chk(bias, "bias of the values to mix in", torch.float32, (first.shape[1],))
+            mix_bias = c_void_p(bias.data_ptr() + col * 4)
     q_out = torch.empty(M, nq, dk, dtype=dtype, device=proj.device)
     check(fn("snk_split_prepare")(
         _ptr(proj), width, q_off, k_off, v_off, _ptr(proj_bias), _ptr(q_gamma), _ptr(k_gamma), g32,
@@ -1682,7 +1885,7 @@ def split_prepare(proj, q_off, k_off, v_off, q_gamma, k_gamma, eps, inv_freq, ro
         float(eps),
         _ptr(inv_freq), rot, float(rot_mult), _ptr(positions), _ptr(row_seg), _ptr(block_table),
         block_table.shape[1], page_size, _ptr(kpool), _ptr(vpool), _ptr(q_out), M, nq, nkv * maps, nkv, dk, dv,
-        int(write_kv), code_of(dtype), _stream()), "split_prepare",
+        int(write_kv), mix_ptr, mix_ld, mix_bias, float(lam), code_of(dtype), _stream()), "split_prepare",
         work=lambda: (2 * M * need * proj.element_size(), 0))
     return q_out
 
@@ -1715,7 +1918,7 @@ def reach_code(window=None, block=None) -> int:
 def split_attention(q, kpool, vpool, block_table, page_size, positions, row_seg, scale, *, maps=1, window=None,
                     bias=None, tiles=None, tile_rows=1, out_dtype=None, out=None, num_chunks=1, scratch=None,
                     chunk=SPLIT_ATTENTION_CHUNK, block=None, head_scale=None, sink=None, keep=0, slopes=None,
-                    gate=None, gate_col=0):
+                    gate=None, gate_col=0, softcap=None):
     """Causal attention of q [M, nq, dk] (nq = heads * maps) over keys [pages, nkv, page_size, maps*dk] and
     values [pages, nkv, page_size, dv]; query head (h, map) reads the key at offset map*dk of its kv head.
     ``window``: the last ``window`` keys only; ``block``: the keys of the query's own block of ``block``
@@ -1728,7 +1931,8 @@ def split_attention(q, kpool, vpool, block_table, page_size, positions, row_seg,
     ``attention_scratch_bytes`` says).  ``keep``: beside its window a query also reaches the positions below
     ``keep`` (``split_attention_chunks`` counts a row's chunks then).  ``slopes`` float [nq] (instead of
     ``bias``): slopes[head] * (i - j) is taken off the scaled score.  ``gate`` [M, width] in the compute dtype:
-    head h's output is multiplied by sigmoid(gate[m, gate_col + h]).  Scores, weights and sums are float;
+    head h's output is multiplied by sigmoid(gate[m, gate_col + h]).  ``softcap`` c: the scaled score becomes
+    c * tanh(score / c), ahead of bias and slopes.  Scores, weights and sums are float;
     returns [M, nq, dv] in ``out_dtype`` (float32 or the compute dtype)."""
     M, nq, dk = q.shape
     dtype = q.dtype
@@ -1799,7 +2003,7 @@ def split_attention(q, kpool, vpool, block_table, page_size, positions, row_seg,
         _ptr(row_seg), _ptr(tiles), n_tiles, int(tile_rows), _ptr(out), int(out_dtype == torch.float32 and dtype != torch.float32),
         nq, nkv, int(maps), dk, dv, reach, float(scale), _ptr(bias if slopes is None else slopes),
         -1 if slopes is not None else (bias.shape[1] if bias is not None else 0), _ptr(head_scale), _ptr(sink),
-        keep, gate_ptr, gate_ld, int(chunk), num_chunks, _ptr(scratch),
+        keep, float(softcap or 0.0), gate_ptr, gate_ld, int(chunk), num_chunks, _ptr(scratch),
         code_of(dtype), _stream()), "split_attention", work=work)
     if num_chunks > 1:
         check(fn("snk_attention_merge_gated")(_ptr(scratch), _ptr(positions), _ptr(out), M, nq, dv, reach, keep,
@@ -1962,6 +2166,8 @@ def streams_norm(streams, weight, groups, eps, dtype, *, init=None, update: Stre
             y = y.dense()                  # a factor or a gate per row: forms this kernel does not apply itself
         if isinstance(y, DeltaSum):
             da, y = y.a, y.b
+        if isinstance(y, ExpertSum) and y.x is not None:
+            y = y.dense()                  # identity experts' pairs have no rows
         if isinstance(y, ExpertSum):
             moe = y
             _chk(moe.y, "expert outputs", torch.float32)

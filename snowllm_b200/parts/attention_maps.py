@@ -1,7 +1,7 @@
 """Windowed grouped-query attention mixers whose keys and values have widths of their own
 (csrc/attention_split.cu): keys of ``head_dim``, values of ``v_head_dim``, kept in two pools.
 
-Five kinds are built on one class:
+Six kinds are built on one class:
 
 * ``bias_attention``: one softmax map per head; a learned bias is added to the scaled score, chosen by
   head and by a bucket of the distance i - j (``DistanceBuckets``).  No rotation.
@@ -27,6 +27,9 @@ Five kinds are built on one class:
   reachable at their true positions; one more term 1 in the softmax's denominator (``one_more``: a sink whose
   score is 0 and which has no value); each head's output times sigmoid of the head's own logit from a gate
   projection [heads, hidden] that reads the mixer's input.
+
+* ``rotary_attention``: causal, biased projections, optional per-head norms, rotary positions, optionally a cap on
+  the scores and values mixed with those of the first layer that mixes (``RotaryAttention``).
 
 The first two: per-head RMS norm of q and k with one weight of ``head_dim`` shared by all heads (and maps), before
 the rotation; ``window`` keeps the last ``window`` keys.  Scores, softmax weights and the per-head
@@ -120,6 +123,7 @@ class MapsAttention(Part):
     norm_weights = True        # the per-head norm of q and k has a weight (False: the plain root mean square)
     whole_norm = False         # True: ONE root mean square over all heads of q (of k), weights of that size
     keep_first = 0             # positions at the sequence's start that stay reachable beside the window
+    softcap = None             # c: a scaled score s becomes c * tanh(s / c)
 
     def __init__(self, dtype, names, *, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int,
                  v_head_dim: int, scale: float, qk_norm_eps: float | None, window: int | None = None,
@@ -218,7 +222,7 @@ class MapsAttention(Part):
                                   self.num_kv_heads, self.maps, self.head_dim, self.v_head_dim,
                                   write_kv=owns_cache, proj_bias=self.proj_bias,
                                   plain_norm=self.qk_norm_eps is not None and not self.norm_weights,
-                                  whole_norm=self.whole_norm)
+                                  whole_norm=self.whole_norm, value_mix=self._value_mix(ctx, rows, v_off))
         ctx.tap("attention_q", q)
         if self._prompt_kernel_ok(ctx, q, cache, out_dtype):
             # prompt portions on the tcgen05 kernel; the rows of short segments (decoded tokens beside them) below
@@ -245,15 +249,15 @@ class MapsAttention(Part):
         keys and values alike, a mask and a bias it knows (causal, a window with or without kept first keys, a
         slope per head, a sink per head, a gate per head)."""
         return (self.maps == 1 and self.head_dim == 64 and self.v_head_dim == 64 and self.bias is None
-                and self.block is None and self.head_scale is None and out_dtype == torch.bfloat16
-                and kernels.attention_prefill_tc_ok(q, cache.page_size)
+                and self.block is None and self.head_scale is None and self.softcap is None
+                and out_dtype == torch.bfloat16 and kernels.attention_prefill_tc_ok(q, cache.page_size)
                 and max(ctx.host_seg_len) >= plan.PREFILL_MIN_ROWS)
 
     def _decode_kernel_ok(self, q, cache, out_dtype) -> bool:
         """Whether rows that stand alone go to the TMA decode kernel: bfloat16, one map, heads of 64 or 128 for
         keys and values alike, up to 16 heads per kv head, a mask and a bias it knows."""
         return (self.maps == 1 and self.head_dim == self.v_head_dim and self.head_dim in kernels.PREFILL_HEAD_DIMS
-                and self.bias is None and self.block is None and self.head_scale is None
+                and self.bias is None and self.block is None and self.head_scale is None and self.softcap is None
                 and out_dtype == torch.bfloat16 and q.dtype == torch.bfloat16
                 and self.nq // self.num_kv_heads <= kernels.DECODE_MMA_MAX_GROUP
                 and kernels.DECODE_TMA and kernels.decode_tma_page_ok(cache.page_size))
@@ -304,9 +308,14 @@ class MapsAttention(Part):
                                       out_dtype=out_dtype, num_chunks=num_chunks, scratch=scratch, chunk=chunk,
                                       block=self.block, head_scale=self.head_scale, sink=self.sink,
                                       keep=self.keep_first, slopes=self.slopes,
-                                      gate=proj if self._gate_in_kernel() else None, gate_col=g_off)
+                                      gate=proj if self._gate_in_kernel() else None, gate_col=g_off,
+                                      softcap=self.softcap)
         ctx.tap("attention_o", out)
         return out
+
+    def _value_mix(self, ctx, rows, v_off):
+        """What ``kernels.split_prepare`` mixes into this layer's values (None: nothing)."""
+        return None
 
     def _convolved(self, ctx, proj, cache):
         """(the paged view, the rows split_prepare reads): a kind whose projections pass something on their
@@ -507,6 +516,60 @@ class ConvGateAttention(MapsAttention):
         return linear(out.view(ctx.M, -1), self.wo, out_dtype=torch.float32)
 
 
+class RotaryAttention(MapsAttention):
+    """One map per head; projections with biases; per-head RMS norm of q and k (``qk_norm_eps`` None: none) before the
+    rotation; ``softcap`` c on the scaled scores; and values that go over into those of an earlier layer: with
+    ``value_mix`` "first" the layer leaves its values in the step's memo, with "mix" it caches (1 - lambda) v +
+    lambda v_first (lambda a learned number, ``value_mix`` among its tensors in either role)."""
+    libraries = MapsAttention.libraries + ("attention_tc", "attention_mma")
+    VALUES = "first_values"            # the memo key under which the first mixing layer's values are found
+
+    def __init__(self, dtype, names, *, softcap: float | None = None, value_mix: str | None = None, biased: bool = True,
+                 **kw):
+        super().__init__(dtype, names, **kw)
+        if softcap is not None and not softcap > 0:
+            raise ConfigError(f"a score cap of {softcap}: want a positive number")
+        if value_mix not in (None, "first", "mix"):
+            raise ConfigError(f"value_mix={value_mix!r} (known: first, mix)")
+        if self.reads_cache and value_mix is not None:
+            raise ConfigError("a layer that reads another layer's cache has no values to mix")
+        self.softcap, self.value_role, self.biased = softcap, value_mix, biased
+        self.value_lambda = 0.0
+
+    def declare(self, has):
+        n, dk, dv = self.names, self.head_dim, self.v_head_dim
+        specs = super().declare(has)
+        if self.biased:
+            specs += [TensorSpec("q_bias", n["q_bias"], (self.num_heads * dk,), INIT_BIAS, KEEP_F32),
+                      TensorSpec("k_bias", n["k_bias"], (self.num_kv_heads * dk,), INIT_BIAS, KEEP_F32),
+                      TensorSpec("v_bias", n["v_bias"], (self.num_kv_heads * dv,), INIT_BIAS, KEEP_F32)]
+        if self.value_role is not None:
+            specs.append(TensorSpec("value_mix", n["value_mix"], (), INIT_BIAS, KEEP_F32))
+        return specs
+
+    def bind(self, tensors):
+        super().bind(tensors)
+        if self.biased:
+            bias = torch.cat([tensors[k].float() for k in ("q_bias", "k_bias", "v_bias")])
+            self.proj_bias = torch.cat((bias, bias.new_zeros(self.w_in.shape[0] - bias.numel()))).contiguous()
+        if self.value_role == "mix":
+            self.value_lambda = float(tensors["value_mix"])
+
+    def _value_mix(self, ctx, rows, v_off):
+        if self.value_role == "first":
+            ctx.memo[self.VALUES] = (rows, v_off, self.proj_bias)
+        elif self.value_role == "mix":
+            if self.VALUES not in ctx.memo:
+                raise KernelError("a layer whose values mix needs an earlier layer that leaves its values")
+            return (*ctx.memo[self.VALUES], self.value_lambda)
+        return None
+
+    def forward(self, ctx, x, cache, owns_cache=True):
+        _, out = self._attend(ctx, x, cache, owns_cache, self.dtype)
+        return linear(out.view(ctx.M, -1), self.wo, out_dtype=torch.float32)
+
+
+register_mixer("rotary_attention", RotaryAttention)
 register_mixer("sink_attention", SinkAttention)
 register_mixer("slope_attention", SlopeAttention)
 register_mixer("conv_gate_attention", ConvGateAttention)

@@ -12,7 +12,10 @@ their outputs is left to the norm that follows (``kernels.DeltaSum``).
 
 ``hyper``: the stream is kept as S streams (hyper-connections).  Sublayer q reads u = sum_s in_q[s] X[s]
 through its norm and leaves y; then X'[t] = sum_s mix_q[s, t] X[s] + out_q[t] y for all t at once.  The
-update stays pending (``kernels.StreamsDelta``) until the next norm applies it in its own kernel."""
+update stays pending (``kernels.StreamsDelta``) until the next norm applies it in its own kernel.
+
+``sandwich``: x += post(gate * mixer(pre(x))); x += post(gate * ffn(pre(x))), a norm on both sides of each
+sublayer, a gate per element, and a learned average over all layers' results so far."""
 from __future__ import annotations
 
 import torch
@@ -21,8 +24,9 @@ from ..errors import ConfigError
 from ..ops import kernels
 from ..trace import span
 from .base import Part
-from .registry import register_block
-from .spec import KEEP_F32, TensorSpec
+from ..ops import linear
+from .registry import lookup, register_block
+from .spec import INIT_BIAS, KEEP_F32, TensorSpec
 
 
 class PreNormBlock:
@@ -257,6 +261,113 @@ class HyperBlock:
         return pending
 
 
+class OutputGate(Part):
+    """A gate per element on a sublayer's output, sigmoid(W h + b) of the sublayer's input h: the logits W h come from
+    one product in the compute dtype, bias and sigmoid are applied in float by the norm that adds the output."""
+    libraries = ("gemm", "gemm_skinny", "gemm_tc", "gemm_tc2")
+
+    def __init__(self, dtype, names, *, hidden_size: int):
+        super().__init__(dtype, names)
+        self.hidden_size = hidden_size
+        self.weight = self.bias = None
+
+    def declare(self, has):
+        W, n = self.hidden_size, self.names
+        return [TensorSpec("weight", n["weight"], (W, W)), TensorSpec("bias", n["bias"], (W,), INIT_BIAS, KEEP_F32)]
+
+    def bind(self, tensors):
+        self.weight, self.bias = tensors["weight"], tensors["bias"]
+
+    def forward(self, ctx, h):
+        """What a ``kernels.NormedDelta`` takes as its gate."""
+        return linear(h, self.weight), 0, self.bias
+
+
+class DepthAverage(Part):
+    """The learned weights of layer ``index``'s average over the embedding output and the layers' results so far:
+    ``index`` + 2 numbers, kept in float."""
+
+    def __init__(self, dtype, names, *, index: int):
+        super().__init__(dtype, names)
+        self.index = int(index)
+        self.weight = None
+
+    def declare(self, has):
+        return [TensorSpec("weight", self.names["weight"], (self.index + 2,), INIT_BIAS, KEEP_F32)]
+
+    def bind(self, tensors):
+        self.weight = tensors["weight"]
+
+
+class SandwichBlock:
+    """A norm before and after each sublayer: x += post(gate * sublayer(pre(x))), the gate per element sigmoid(W h +
+    b) of h = pre(x) (``gates`` None: no gate).  ``average`` = {"index", "layers", "name"}: what goes on to the next
+    layer is sum_j a[j] X_j over the embedding output X_0 and the layers' results X_1 .. X_(index + 1), which lie in
+    the step's memo.  A sublayer's update stays pending (``kernels.NormedDelta``) for the norm that follows, in this
+    layer, the next one or the model's end: gate, output norm, residual sum, average and that norm are one kernel."""
+    libraries = ("sandwich",)
+
+    def __init__(self, mixer, ffn, mixer_norm, ffn_norm, *, dtype=torch.float32, hidden_size: int, post_norms, gates=None,
+                 average: dict | None = None):
+        self.mixer, self.ffn, self.mixer_norm, self.ffn_norm = mixer, ffn, mixer_norm, ffn_norm
+        sublayers = 1 if ffn is None else 2
+        if len(post_norms) != sublayers or (gates is not None and len(gates) != sublayers):
+            raise ConfigError(f"a layer of {sublayers} sublayers needs as many output norms and gates")
+        for norm in (mixer_norm, ffn_norm):
+            if norm is not None and not getattr(norm, "fusable_rms", False):
+                raise ConfigError(f"a sandwich layer needs RMS norms, not {type(norm).__name__}")
+        self.post = [lookup("norm", s.kind)(torch.float32, s.names, **dict(s.params)) for s in post_norms]
+        self.gates = [OutputGate(dtype, n, hidden_size=hidden_size) for n in gates] if gates is not None else None
+        self.average, self.layers = None, 0
+        if average is not None:
+            self.average = DepthAverage(dtype, dict(weight=average["name"]), index=average["index"])
+            self.layers = int(average["layers"])
+        self._names = tuple(f"{what}:{type(part).__name__}" for what, part in
+                            (("norm", mixer_norm), ("mixer", mixer), ("norm", ffn_norm), ("ffn", ffn)))
+
+    def parts(self):
+        own = tuple(p for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn) if p is not None)
+        return own + tuple(self.post) + tuple(self.gates or ()) + ((self.average,) if self.average else ())
+
+    def _pending(self, ctx, q: int, y, h, last: bool, history):
+        gate = self.gates[q].forward(ctx, h) if self.gates is not None else None
+        post = self.post[q]
+        kept = dict(history=history, index=self.average.index + 1, average=self.average.weight) \
+            if last and self.average is not None else {}
+        return kernels.NormedDelta(y, gate=gate, weight=post.weight, eps=post.eps, **kept)
+
+    def forward(self, ctx, residual, delta, cache, owns_cache=True):
+        history = None
+        if self.average is not None:
+            key = ("depth_history", id(residual))
+            history = ctx.memo.get(key)
+            if history is None:
+                if self.average.index != 0 or delta is not None:
+                    raise ConfigError("a depth average starts at the model's first layer")
+                history = ctx.memo[key] = torch.empty(self.layers + 1, *residual.shape, dtype=torch.float32,
+                                                      device=residual.device)
+                delta = kernels.NormedDelta(None, history=history, index=0)     # X_0, the embedding output
+        with span(self._names[0]):
+            h = self.mixer_norm.forward(ctx, residual, delta)
+        ctx.tap("mixer_in", h)
+        with span(self._names[1]):
+            y = self.mixer.forward(ctx, h, cache, owns_cache)
+        ctx.tap("mixer_out", y)
+        pending = self._pending(ctx, 0, y, h, self.ffn is None, history)
+        if self.ffn is not None:
+            with span(self._names[2]):
+                h = self.ffn_norm.forward(ctx, residual, pending)
+            ctx.tap("ffn_in", h)
+            with span(self._names[3]):
+                y = self.ffn.forward(ctx, h)
+            ctx.tap("ffn_out", y)
+            pending = self._pending(ctx, 1, y, h, True, history)
+        if ctx.taps is not None:
+            ctx.tap("layer_out", pending.total(residual))
+        return pending
+
+
+register_block("sandwich", SandwichBlock)
 register_block("prenorm", PreNormBlock)
 register_block("hyper", HyperBlock)
 register_block("parallel", ParallelBlock)

@@ -6,19 +6,25 @@ import torch
 
 from ..ops import kernels, linear
 from .base import Part
-from .registry import register_embedding, register_head
+from .registry import lookup, register_embedding, register_head
 from ..errors import ConfigError
-from .spec import SlotStateSpec, TensorSpec
+from .spec import PartSpec, SlotStateSpec, TensorSpec
 
 
 class Embedding(Part):
     libraries = ("elementwise",)
 
-    def __init__(self, dtype, names, *, vocab_size: int, hidden_size: int, scale: float = 1.0):
-        """``scale``: a constant that multiplies every row on its way into the stream."""
+    def __init__(self, dtype, names, *, vocab_size: int, hidden_size: int, scale: float = 1.0,
+                 norm: PartSpec | None = None):
+        """``scale``: a constant that multiplies every row on its way into the stream; ``norm``: a norm the rows pass
+        before they enter it (in float, like the stream)."""
         super().__init__(dtype, names)
         self.vocab_size, self.hidden_size, self.scale = vocab_size, hidden_size, float(scale)
         self.weight = None
+        self.norm = lookup("norm", norm.kind)(torch.float32, norm.names, **dict(norm.params)) if norm else None
+
+    def parts(self):
+        return (self.norm,) if self.norm is not None else ()
 
     def declare(self, has):
         return [TensorSpec("weight", self.names["weight"], (self.vocab_size, self.hidden_size))]
@@ -31,7 +37,8 @@ class Embedding(Part):
 
     def forward(self, ctx):
         """The float residual stream [M, H] of the step's tokens."""
-        return kernels.embedding(ctx.token_ids, self.weight, pending=ctx.pending_tokens, scale=self.scale)
+        x = kernels.embedding(ctx.token_ids, self.weight, pending=ctx.pending_tokens, scale=self.scale)
+        return x if self.norm is None else self.norm.forward(ctx, x)
 
 
 class PairHashEmbedding(Embedding):

@@ -13,7 +13,11 @@ one more expert of the same form (a width and a limit of its own) that every tok
 added (the sum is left as a ``kernels.DeltaSum``); with ``shared["row_gate"]`` its output is first multiplied
 by sigmoid(w_sg . x), one number per token (tensor ``shared_row_gate`` [1, hidden]).  ``scoring``
 "softmax_picked": the router's logits, plus the bias ``expert_bias`` which is then a part of the logit, pick
-the k largest, and the weights are the softmax over the picked logits alone."""
+the k largest, and the weights are the softmax over the picked logits alone.  With ``scoring`` "softmax" an
+``expert_bias`` is a correction that only chooses.  ``groups`` (count, keep): the router's outputs form equal groups
+of neighbours, and only experts of the best ``keep`` groups can be chosen.  ``identity``: that many more router
+outputs stand for experts that return their input.  ``gated`` False: an expert is down(act(up x)), ``activation`` one
+of the plain ones (the square of relu among them)."""
 from __future__ import annotations
 
 import torch
@@ -31,21 +35,30 @@ class SigmoidMoE(Part):
     def __init__(self, dtype, names, *, hidden_size: int, intermediate_size: int, num_experts: int,
                  top_k: int, norm_topk_prob: bool, use_expert_bias: bool, routed_scaling_factor: float,
                  scale_input: bool = False, scoring: str = "sigmoid", activation: str = "silu",
-                 limit: float | None = None, shared: dict | None = None):
+                 limit: float | None = None, shared: dict | None = None, gated: bool = True, groups=(1, 1),
+                 identity: int = 0):
         """``scale_input``: a pick's weight multiplies the expert's INPUT (the output is the plain sum of
         expert(w * x) over the picks) instead of its output.  ``shared``: {"intermediate_size", "limit"}."""
         super().__init__(dtype, names)
         if scoring not in kernels.ROUTER_SCORINGS:
             raise ConfigError(f"router scoring {scoring!r} (known: {', '.join(kernels.ROUTER_SCORINGS)})")
-        if activation not in ("silu", "swish_clamp"):
+        if not gated:
+            if activation not in kernels.ACTIVATIONS or scale_input or shared is not None:
+                raise ConfigError(f"ungated experts with activation {activation!r} (known: "
+                                  f"{', '.join(kernels.ACTIVATIONS)}; no scaled input, no shared expert)")
+        elif activation not in ("silu", "swish_clamp"):
             raise ConfigError(f"expert activation {activation!r} (known: silu, swish_clamp)")
         if activation == "swish_clamp" and not (limit and limit > 0):
             raise ConfigError("the clamped activation needs a positive limit")
         if shared is not None and not (activation == "swish_clamp" and shared.get("limit", 0) > 0
                                        and shared.get("intermediate_size", 0) > 0):
             raise ConfigError("a shared expert has the clamped form, with a width and a positive limit of its own")
-        if scoring == "softmax" and use_expert_bias:
-            raise ConfigError("an expert bias goes with sigmoid scores")
+        self.gated, self.groups, self.identity = bool(gated), (int(groups[0]), int(groups[1])), int(identity)
+        if self.identity and gated:
+            raise ConfigError("identity experts go with ungated experts")
+        if self.groups[0] > 128 or (num_experts + self.identity) % self.groups[0]:
+            raise ConfigError(f"{num_experts + self.identity} router outputs in {self.groups[0]} groups (up to 128 equal "
+                              f"groups)")
         self.scoring, self.activation, self.limit = scoring, activation, limit
         self.shared = dict(shared) if shared is not None else None
         self.shared_w13 = self.shared_w2 = self.shared_row_gate = None
@@ -54,16 +67,23 @@ class SigmoidMoE(Part):
         self.norm_topk_prob, self.use_expert_bias = norm_topk_prob, use_expert_bias
         self.routed_scaling_factor = routed_scaling_factor
         self.scale_input = scale_input
-        self.router = self.bias = self.w13 = self.w2 = None
+        self.router = self.bias = self.w13 = self.w1 = self.w2 = None
         self._fused = False
         self._ticket = None            # the counter of the one-launch front end (zero between launches)
 
     def declare(self, has):
         H, I, E = self.hidden_size, self.intermediate_size, self.num_experts
         n = self.names
-        specs = [TensorSpec("router", n["router"], (E, H), keep=KEEP_SMALL)]
+        outputs = E + self.identity
+        specs = [TensorSpec("router", n["router"], (outputs, H), keep=KEEP_SMALL)]
         if self.use_expert_bias:
-            specs.append(TensorSpec("expert_bias", n["expert_bias"], (E,), INIT_BIAS, KEEP_F32))
+            specs.append(TensorSpec("expert_bias", n["expert_bias"], (outputs,), INIT_BIAS, KEEP_F32))
+        if not self.gated:
+            for e in range(E):
+                p = f"{n['experts']}{e}."
+                specs += [TensorSpec(f"up.{e}", p + n["expert_up"], (I, H)),
+                          TensorSpec(f"down.{e}", p + n["expert_down"], (H, I))]
+            return specs
         self._fused = has(n["fused_gate_up"])
         if self._fused:
             specs += [TensorSpec("gate_up", n["fused_gate_up"], (E, 2 * I, H)),
@@ -86,6 +106,10 @@ class SigmoidMoE(Part):
         E = self.num_experts
         self.router = tensors["router"]
         self.bias = tensors.get("expert_bias") if self.use_expert_bias else None
+        if not self.gated:
+            self.w1 = torch.stack([tensors[f"up.{e}"] for e in range(E)]).contiguous()
+            self.w2 = torch.stack([tensors[f"down.{e}"] for e in range(E)]).contiguous()
+            return
         if self._fused:
             gate, up = tensors["gate_up"].chunk(2, dim=1)
             self.w2 = tensors["down"].contiguous()
@@ -114,7 +138,7 @@ class SigmoidMoE(Part):
 
     def route(self, x):
         return kernels.moe_route(x, self.router, self.bias, self.top_k, self.norm_topk_prob,
-                                 self.routed_scaling_factor, self.scoring)
+                                 self.routed_scaling_factor, self.scoring, self.groups)
 
     def forward_from_residual(self, ctx, residual, delta, norm):
         """The norm that precedes this feed-forward, the router and the sort in one launch, for the few rows
@@ -125,7 +149,7 @@ class SigmoidMoE(Part):
             return None
         if self.scale_input or not kernels.FUSE_ROUTER or not kernels.norm_route_sort_ok(residual, delta, weight, self.router, self.top_k):
             return None
-        if self.scoring != "sigmoid" or self.activation != "silu" or self.shared is not None:
+        if self.scoring != "sigmoid" or self.activation != "silu" or self.shared is not None or self.groups[0] > 1:
             return None
         if self._ticket is None or self._ticket.device != residual.device:
             self._ticket = torch.zeros(1, dtype=torch.int32, device=residual.device)
@@ -138,7 +162,8 @@ class SigmoidMoE(Part):
 
     def forward(self, ctx, x):
         routed = self._experts(ctx, x, *kernels.moe_route_sort(
-            x, self.router, self.bias, self.top_k, self.norm_topk_prob, self.routed_scaling_factor, self.scoring))
+            x, self.router, self.bias, self.top_k, self.norm_topk_prob, self.routed_scaling_factor, self.scoring,
+            self.groups, self.identity))
         if self.shared is None:
             return routed
         act = linear_glu(x, self.shared_w13, self.shared_interleaved, self.activation, self.shared["limit"])
@@ -160,6 +185,12 @@ class SigmoidMoE(Part):
             ctx.tap("moe_route", ids)
             ctx.tap("moe_route_input", x)
         cap = min(M, M * k)          # an expert gets a token at most once
+        if not self.gated:
+            # the pairs of identity experts sort behind the others and own no rows in the products
+            own = offsets[:self.num_experts + 1]
+            act = kernels.act_rows(grouped_linear(x, self.w1, own, M * k, cap, sorted_pair, k), self.activation)
+            y = grouped_linear(act, self.w2, own, M * k, cap, out_dtype=torch.float32)
+            return kernels.ExpertSum(y, pair_pos, weights, x=x if self.identity else None)
         if self.scale_input:
             # the rows in expert order, each times its pick's weight; the outputs are then summed as they are
             xs, weights = kernels.moe_scaled_rows(x, sorted_pair, weights, k)

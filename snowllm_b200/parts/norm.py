@@ -10,7 +10,7 @@ from ..errors import ConfigError
 from ..ops import kernels
 from .base import Part
 from .registry import register_norm
-from .spec import INIT_BIAS, INIT_ONES, KEEP_SMALL, TensorSpec
+from .spec import INIT_BIAS, INIT_ONES, KEEP_F32, KEEP_SMALL, TensorSpec
 
 
 class RMSNorm(Part):
@@ -18,20 +18,25 @@ class RMSNorm(Part):
     fusable_rms = True     # x * rsqrt(mean(x^2) + eps) * weight over the whole width: what a part that fuses
                            # the norm before it into its own first kernel may take over (weight, eps)
 
-    def __init__(self, dtype, names, *, size: int, eps: float):
+    def __init__(self, dtype, names, *, size: int, eps: float, offset: float = 0.0):
+        """``offset``: a constant added to the stored weight (1 for weights stored around zero); the sum is kept in
+        float."""
         super().__init__(dtype, names)
-        self.size, self.eps = size, eps
+        self.size, self.eps, self.offset = size, eps, float(offset)
         self.weight = None
 
     def declare(self, has):
+        if self.offset:
+            return [TensorSpec("weight", self.names["weight"], (self.size,), INIT_BIAS, KEEP_F32)]
         return [TensorSpec("weight", self.names["weight"], (self.size,), INIT_ONES, KEEP_SMALL)]
 
     def bind(self, tensors):
-        self.weight = tensors["weight"]
+        self.weight = tensors["weight"] + self.offset if self.offset else tensors["weight"]
 
     def forward(self, ctx, residual, delta=None, rows=None):
         """``residual += delta`` in float, then the norm of the sum in the compute dtype.  With
-        ``rows`` (int32 row numbers) only those rows come out and the residual stays untouched."""
+        ``rows`` (int32 row numbers) only those rows come out and the residual stays untouched.  A
+        ``kernels.NormedDelta`` is applied with its own norm, gate and depth average."""
         return kernels.add_rmsnorm(residual, delta, self.weight, self.eps, self.dtype, rows=rows)
 
     def add_normed(self, ctx, residual, y):

@@ -96,6 +96,36 @@ class YarnRotaryPosition:
         return self._inv_freq, self.rot_dim
 
 
+class BandedRotaryPosition(RotaryPosition):
+    """Rotary frequencies rescaled by bands of wavelength, as Llama 3.1 does for contexts longer than the ``original``
+    one: with wavelength l = 2 pi / f, a frequency is kept where l < original / high, divided by ``factor`` where l >
+    original / low, and in between goes over linearly in original / l.  ``scaling`` None: the plain table.  Worked out
+    in double precision on the host and kept in float."""
+
+    def __init__(self, *, head_dim: int, theta: float, rot_dim: int | None = None, scaling: dict | None = None):
+        super().__init__(head_dim=head_dim, theta=theta, rot_dim=rot_dim, precise=True)
+        self.scaling = dict(scaling) if scaling else None
+
+    def frequencies(self) -> list:
+        plain = [self.theta ** (-2.0 * i / self.rot_dim) for i in range(self.rot_dim // 2)]
+        return plain if self.scaling is None else [self._rescaled(f, **self.scaling) for f in plain]
+
+    @staticmethod
+    def _rescaled(f: float, factor: float, low: float, high: float, original: float) -> float:
+        turns = original * f / (2.0 * math.pi)             # how often the pair turns over the original context
+        if turns > high:
+            return f
+        if turns < low:
+            return f / factor
+        keep = (turns - low) / (high - low)
+        return (1.0 - keep) * f / factor + keep * f
+
+    def rotary(self, device):
+        if self._inv_freq is None or self._inv_freq.device != torch.device(device):
+            self._inv_freq = torch.tensor(self.frequencies(), dtype=torch.float64).to(torch.float32).to(device)
+        return self._inv_freq, self.rot_dim
+
+
 class NoPosition:
     """No position encoding (the mixer sees order only through its causal mask)."""
 
@@ -107,6 +137,7 @@ class NoPosition:
 
 
 register_position("rope", RotaryPosition)
+register_position("rope_bands", BandedRotaryPosition)
 register_position("none", NoPosition)
 register_position("yarn", YarnRotaryPosition)
 register_position("rope_pairs", PairedRotaryPosition)
