@@ -1,7 +1,7 @@
 """Decode and prefill throughput of the engine at the layer sizes of the LFM2.5 models, random weights.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--config 8b-a1b|dense-1.2b|dense-2.6b]
-    python bench.py --design beledra|zafopel|toderax|kuzupel   (another design beside the closest existing model at equal size; one JSON line)
+    python bench.py --design beledra|zafopel|toderax|kuzupel|gurolix   (another design beside the closest existing model at equal size; one JSON line)
                     [--batch B] [--context C] [--dtype bfloat16|float32] [--impl ours|reference]
 
 Prints ONE JSON line.  Without flags: LFM2.5-8B-A1B sizes, 8 requests at context 8,192.
@@ -225,6 +225,36 @@ def _lfm2_moe_heads64_like(width: int, layers: int, ff: int, vocab: int = 65536)
     return cfg
 
 
+def _gurolix(width: int, layers: int, ff: int, vocab: int = 65536) -> dict:
+    """Gurolix at sizes that resemble a real model's layers: every second layer a state-space mixer (heads of 64, twice
+    the width, a state of 128, B and C shared by groups of heads, 4 taps), between them attention in turns without
+    norms, with rescaled frequencies and scores capped at 30, and with per-head norms (heads of 64, one kv head per
+    four, values mixed with the first layer's); every token goes to 4 of 32 router outputs, 28 experts of ff/8 and 4
+    identity experts, within 2 of 4 groups."""
+    heads = width // 64
+    attn = {"heads": heads, "kv_heads": max(heads // 4, 1), "dim": 64, "vdim": 64, "scale": 0.125, "v_mix": True}
+    capped = dict(attn, softcap=30.0, rot={"dims": 64, "base": 500000.0, "scaling": {
+        "factor": 32.0, "low": 1.0, "high": 4.0, "original": 8192}})
+    normed = dict(attn, rot={"dims": 64, "base": 10000.0})
+    groups = max(width // 256, 1)
+    state = {"heads": width // 32, "vdim": 64, "state": 128, "groups": groups, "norm_groups": groups, "conv": 4}
+    mlp = {"kind": "moe", "expert": {"ff": ff // 8}, "router": {"experts": 28, "identity": 4, "top": 4,
+                                                                "groups": {"count": 4, "keep": 2}}}
+    kinds = [("attention_2", capped), ("mamba2", state), ("attention", normed), ("mamba2", state)]
+    out = [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": mlp} for i in range(layers)]
+    return {"architecture": "Gurolix", "vocab": vocab, "width": width, "norm": {"eps": 1e-5},
+            "layers": json.loads(json.dumps(out))}
+
+
+def _lfm2_moe_alternating_like(width: int, layers: int, ff: int, vocab: int = 65536) -> dict:
+    """The closest existing model at equal size: LFM2 with routed experts at equal width and depth, attention with
+    equal head counts wherever the other design has attention, a short convolution wherever it has a state-space
+    mixer, 4 of 32 experts of ff/8 in every layer but the first, which is dense."""
+    cfg = _lfm2_moe_heads64_like(width, layers, ff, vocab)
+    cfg["layer_types"] = ["conv" if i % 2 else "full_attention" for i in range(layers)]
+    return cfg
+
+
 DESIGN_SIZES = {"w2048-l12": (2048, 12, 8192), "w1024-l6": (1024, 6, 4096)}
 # design -> (its name, its configuration at a size, the closest existing model at that size, what that is)
 DESIGNS = {"beledra": ("Beledra", _beledra, ("lfm2_dense", _lfm2_like),
@@ -236,7 +266,11 @@ DESIGNS = {"beledra": ("Beledra", _beledra, ("lfm2_dense", _lfm2_like),
                        "memory alone, attention with equal head counts where it has a pair, equal expert count and width"),
            "kuzupel": ("Kuzupel", _kuzupel, ("lfm2_moe_heads64", _lfm2_moe_heads64_like),
                        "LFM2 with routed experts at equal width, depth, head count and size (64), expert count and width; "
-                       "its attention sees every key, the design's a window")}
+                       "its attention sees every key, the design's a window"),
+           "gurolix": ("Gurolix", _gurolix, ("lfm2_moe_alternating", _lfm2_moe_alternating_like),
+                       "LFM2 with routed experts at equal width and depth: attention with equal head counts and size where "
+                       "the design has attention, a short convolution where it has a state-space mixer, 32 experts of "
+                       "equal width")}
 
 
 def design_compare(a) -> dict:

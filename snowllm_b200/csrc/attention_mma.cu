@@ -812,7 +812,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const __
                             float* __restrict__ part_o, float* __restrict__ part_ml, int nh, int nkv,
                             int window, int num_chunks, float scale_log2, int keep,
                             const float* __restrict__ slopes, const float* __restrict__ sink,
-                            const bf16* __restrict__ gate, long long gate_ld) {
+                            const bf16* __restrict__ gate, long long gate_ld, float cap_in) {
   // the map is a kernel parameter: fetching it does not have to wait for the kernel in front
   if (threadIdx.x == 0) {
     asm volatile("prefetch.tensormap [%0];" ::"l"(reinterpret_cast<uint64_t>(&map_kv)) : "memory");
@@ -822,6 +822,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const __
     keep = 0;
     slopes = sink = nullptr;
     gate = nullptr;
+    cap_in = 0.f;
   }
   pdl_begin();
   constexpr int CH = HD / 8, KT = HD / 16, NT = HD / 8, PANELS = HD / 64;
@@ -945,6 +946,12 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const __
         fa_mma(s[2 * n + 1], qf[k][0], qf[k][1], qf[k][2], qf[k][3], b2, b3);
       }
     }
+    if (cap_in > 0.f) {                                   // tanh(score / cap) takes the score's place: 1 - 2 / (e^(2z) + 1)
+#pragma unroll
+      for (int i = 0; i < FA_BK / 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) s[i][j] = 1.f - __fdividef(2.f, exp2f(fminf(s[i][j] * cap_in, 60.f)) + 1.f);
+    }
     float mx[2] = {-INFINITY, -INFINITY};
     float slope2[2] = {0.f, 0.f};                         // this thread's two rows' slopes, in units of log 2
     if (slopes) {
@@ -1058,7 +1065,7 @@ static int fd_launch(const void* q, const void* pool, const void* vpool, long lo
                      int max_pages, int page_size, const int* positions, const int* row_seg,
                      const int* row_list, void* out, void* scratch, int M, int nh, int nkv,
                      int hd, int window, int num_chunks, float scale, int keep, const float* slopes,
-                     const float* sink, const void* gate, long long gate_ld, cudaStream_t stream) {
+                     const float* sink, const void* gate, long long gate_ld, float softcap, cudaStream_t stream) {
   if (M <= 0) return 0;
   if (keep < 0 || (keep > 0 && window <= 0)) return SNK_ERR_SIZE;
   if (nkv <= 0 || nh % nkv || nh / nkv > 16 || nkv > 65535 || num_chunks < 1 || num_chunks > 65535)
@@ -1077,9 +1084,11 @@ static int fd_launch(const void* q, const void* pool, const void* vpool, long lo
     rc = tensor_map(vpool, num_pages * nkv * page_size, hd, page_size, 64, &map_v);
     if (rc) return rc;
   }
-  const bool extra = vpool || keep || slopes || sink || gate;
+  const bool extra = vpool || keep || slopes || sink || gate || softcap > 0.f;
   const bf16* gp = static_cast<const bf16*>(gate);
-  const float scale_log2 = scale * 1.4426950408889634f;
+  // with a cap c the scores become c tanh(scale q . k / c): the tangent's argument, and what then takes the scale's place
+  const float cap_in = softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f;
+  const float scale_log2 = (softcap > 0.f ? softcap : scale) * 1.4426950408889634f;
   dim3 grid(M, nkv, num_chunks);
   const size_t smem = 1024 + (size_t)2 * (hd / 64) * FD_CHUNK * 128 + (size_t)16 * hd * 2;
   float* part_o = static_cast<float*>(scratch);
@@ -1092,7 +1101,8 @@ static int fd_launch(const void* q, const void* pool, const void* vpool, long lo
                          (int)smem);                                                                             \
     snk_launch(attention_decode_tma_kernel<HD_, EXTRA_>, dim3(grid), dim3(FA_WARPS * 32), smem, stream, map,     \
                map_v, k_mul, v_add, qp, block_table, max_pages, page_size, positions, row_seg, row_list, op,     \
-               part_o, part_ml, nh, nkv, window, num_chunks, scale_log2, keep, slopes, sink, gp, gate_ld);       \
+               part_o, part_ml, nh, nkv, window, num_chunks, scale_log2, keep, slopes, sink, gp, gate_ld,        \
+               cap_in);                                                                                          \
   } while (0)
   if (hd == 64) {
     if (extra) FD_LAUNCH(64, true);
@@ -1111,22 +1121,22 @@ SNK_API int snk_attention_decode_tma(const void* q, const void* pool, long long 
                                      const int* row_list, void* out, void* scratch, int M, int nh, int nkv,
                                      int hd, int window, int num_chunks, float scale, cudaStream_t stream) {
   return fd_launch(q, pool, nullptr, num_pages, block_table, max_pages, page_size, positions, row_seg, row_list, out,
-                   scratch, M, nh, nkv, hd, window, num_chunks, scale, 0, nullptr, nullptr, nullptr, 0, stream);
+                   scratch, M, nh, nkv, hd, window, num_chunks, scale, 0, nullptr, nullptr, nullptr, 0, 0.f, stream);
 }
 
 // The same over keys and values in pools of their own [pages, nkv, page_size, hd], with kept first keys (a row's
 // chunks are then counted as chunk_keys does, and so must the merge), a slope and a sink per head (float [nh])
 // and a gate per (row, head) (bfloat16, gate[m * gate_ld + head]; applied here when there is one chunk).
-// row_list (may be null): the M rows of the batch to serve, when not all of them.
+// softcap c > 0: the scaled score becomes c tanh(score / c).  row_list (may be null): the M rows of the batch to serve, when not all of them.
 SNK_API int snk_attention_decode_tma_split(const void* q, const void* kpool, const void* vpool, long long num_pages,
                                            const int* block_table, int max_pages, int page_size,
                                            const int* positions, const int* row_seg, const int* row_list, void* out,
                                            void* scratch, int M, int nh, int nkv, int hd, int window, int num_chunks,
                                            float scale, int keep, const float* slopes, const float* sink,
-                                           const void* gate, long long gate_ld, cudaStream_t stream) {
+                                           const void* gate, long long gate_ld, float softcap, cudaStream_t stream) {
   if (!vpool) return SNK_ERR_SIZE;
   return fd_launch(q, kpool, vpool, num_pages, block_table, max_pages, page_size, positions, row_seg, row_list, out,
-                   scratch, M, nh, nkv, hd, window, num_chunks, scale, keep, slopes, sink, gate, gate_ld, stream);
+                   scratch, M, nh, nkv, hd, window, num_chunks, scale, keep, slopes, sink, gate, gate_ld, softcap, stream);
 }
 
 // Queue copies of the two status words (decode, prompt) into ``host`` (pinned host memory, two ints) on

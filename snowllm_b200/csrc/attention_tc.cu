@@ -46,7 +46,9 @@
 //   window's first tile are walked first, in ascending order;
 //   `slopes`: slope[head] * (p - kp) is taken off the scaled score;
 //   `sink`: one more term exp(sink[head]) in the row's sum, without a key or a value (the row starts from it);
-//   `gate`: the head's output times sigmoid(gate[row * gate_ld + head]).
+//   `gate`: the head's output times sigmoid(gate[row * gate_ld + head]);
+//   `softcap` c: the scaled score becomes c tanh(score / c), ahead of slope and mask (a variant of its own: it costs
+//   one exponential and a quarter of a reciprocal more per score, where the plain softmax costs one exponential).
 #include "tcgen05.cuh"
 
 #define AT_BQ 128
@@ -151,14 +153,31 @@ __device__ __forceinline__ float at_exp2(float x) {
 }
 
 // EXTRA false: the kernel without the options (they cost registers that the plain walk has no room for).
-template <bool EXTRA>
+// Four tanh(z) in place of four raw scores r, z = r * k / (2 log2 e): 1 - 2 / (e^(2z) + 1) with one reciprocal for the
+// four (the exponent is cut at 30, where the tangent is 1 to within 2e-9, so the product of four stays finite).
+__device__ __forceinline__ void at_tanh4(uint32_t (&r)[32], int i, float k) {
+  float a[4];
+#pragma unroll
+  for (int e = 0; e < 4; ++e) a[e] = at_exp2(fminf(__uint_as_float(r[i + e]) * k, 30.f)) + 1.f;
+  const float ab = a[0] * a[1], cd = a[2] * a[3];
+  float inv;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(inv) : "f"(ab * cd));
+  const float rab = -2.f * inv * cd, rcd = -2.f * inv * ab;
+  r[i] = __float_as_uint(fmaf(rab, a[1], 1.f));
+  r[i + 1] = __float_as_uint(fmaf(rab, a[0], 1.f));
+  r[i + 2] = __float_as_uint(fmaf(rcd, a[3], 1.f));
+  r[i + 3] = __float_as_uint(fmaf(rcd, a[2], 1.f));
+}
+
+template <bool EXTRA, bool CAP>
 __global__ void __launch_bounds__(AT_THREADS, 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                             const __grid_constant__ CUtensorMap map_v, int k_mul, int v_add,
                             const int* __restrict__ block_table, int max_pages, int page_size,
                             const int* __restrict__ tiles, int n_tiles, bf16* __restrict__ out, int nh, int nkv,
                             int window, float scale_log2, int keep, const float* __restrict__ slopes,
-                            const float* __restrict__ sink, const bf16* __restrict__ gate, long long gate_ld) {
+                            const float* __restrict__ sink, const bf16* __restrict__ gate, long long gate_ld,
+                            float cap_in) {
   if (!EXTRA) {
     keep = 0;
     slopes = sink = nullptr;
@@ -349,6 +368,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&sh->s_empty);
+      if constexpr (CAP) {                               // cap_in: q . k -> 2 log2(e) score / cap; scale_log2: cap log2(e)
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+          for (int i = 0; i < 32; i += 4) at_tanh4(r[c], i, cap_in);
+      }
       if (slopes) {                                      // the distance penalty, before the scale: s - (slope / scale) (p - kp)
         const float base = slope_q * (float)(k0 - pos);
 #pragma unroll
@@ -486,7 +511,7 @@ static bool at_page_ok(int page_size) {
 static int at_launch(const void* q, long long M, const void* pool, const void* vpool, long long num_pages,
                      const int* block_table, int max_pages, int page_size, const int* tiles, int n_tiles, void* out,
                      int nh, int nkv, int hd, int window, float scale, int keep, const float* slopes,
-                     const float* sink, const void* gate, long long gate_ld, cudaStream_t stream) {
+                     const float* sink, const void* gate, long long gate_ld, float softcap, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (nkv <= 0 || nh % nkv || nh > 65535 || M <= 0) return SNK_ERR_SIZE;
   if (hd != AT_HD || !at_page_ok(page_size) || num_pages <= 0) return SNK_ERR_SIZE;
@@ -509,19 +534,29 @@ static int at_launch(const void* q, long long M, const void* pool, const void* v
   const size_t smem = (size_t)(AT_KSTAGES + AT_VSTAGES) * AT_KV_BYTES + AT_P_BYTES + sizeof(AtShared);
   static bool configured = false;
   if (!configured) {
-    cudaFuncSetAttribute(attention_prefill_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    cudaFuncSetAttribute(attention_prefill_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaFuncSetAttribute(attention_prefill_tc_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaFuncSetAttribute(attention_prefill_tc_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaFuncSetAttribute(attention_prefill_tc_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaFuncSetAttribute(attention_prefill_tc_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     configured = true;
   }
-  if (keep || slopes || sink || gate)
-    snk_launch(attention_prefill_tc_kernel<true>, dim3(n_tiles, nh), dim3(AT_THREADS), smem, stream, map_q, map_kv,
-               map_v, k_mul, v_add, block_table, max_pages, page_size, tiles, n_tiles, static_cast<bf16*>(out), nh,
-               nkv, window, scale * 1.4426950408889634f, keep, slopes, sink, static_cast<const bf16*>(gate), gate_ld);
-  else
-    snk_launch(attention_prefill_tc_kernel<false>, dim3(n_tiles, nh), dim3(AT_THREADS), smem, stream, map_q, map_kv,
-               map_v, k_mul, v_add, block_table, max_pages, page_size, tiles, n_tiles, static_cast<bf16*>(out), nh,
-               nkv, window, scale * 1.4426950408889634f, 0, static_cast<const float*>(nullptr),
-               static_cast<const float*>(nullptr), static_cast<const bf16*>(nullptr), 0LL);
+  const float log2e = 1.4426950408889634f;
+  const float scale_log2 = softcap > 0.f ? softcap * log2e : scale * log2e;      // of what enters the softmax
+  const float cap_in = softcap > 0.f ? 2.f * log2e * scale / softcap : 0.f;
+#define AT_LAUNCH(EXTRA_, CAP_)                                                                                  \
+  snk_launch(attention_prefill_tc_kernel<EXTRA_, CAP_>, dim3(n_tiles, nh), dim3(AT_THREADS), smem, stream, map_q, \
+             map_kv, map_v, k_mul, v_add, block_table, max_pages, page_size, tiles, n_tiles,                     \
+             static_cast<bf16*>(out), nh, nkv, window, scale_log2, keep, slopes, sink,                           \
+             static_cast<const bf16*>(gate), gate_ld, cap_in)
+  const bool extra = keep || slopes || sink || gate;
+  if (softcap > 0.f) {
+    if (extra) AT_LAUNCH(true, true);
+    else AT_LAUNCH(false, true);
+  } else {
+    if (extra) AT_LAUNCH(true, false);
+    else AT_LAUNCH(false, false);
+  }
+#undef AT_LAUNCH
   SNK_LAUNCH_CHECK();
   return 0;
 }
@@ -531,21 +566,21 @@ SNK_API int snk_attention_prefill_tc(const void* q, long long M, const void* poo
                                      int n_tiles, void* out, int nh, int nkv, int hd, int window, float scale,
                                      cudaStream_t stream) {
   return at_launch(q, M, pool, nullptr, num_pages, block_table, max_pages, page_size, tiles, n_tiles, out, nh, nkv,
-                   hd, window, scale, 0, nullptr, nullptr, nullptr, 0, stream);
+                   hd, window, scale, 0, nullptr, nullptr, nullptr, 0, 0.f, stream);
 }
 
 // The same with keys [pages, nkv, page_size, 64] and values [pages, nkv, page_size, 64] in pools of their own,
 // kept first keys, a distance slope and a sink per head (float [nh]) and a gate per (row, head) (bfloat16,
-// gate[row * gate_ld + head]); each of them may be off (0 or null).
+// gate[row * gate_ld + head]) and a cap on the scaled scores; each of them may be off (0 or null).
 SNK_API int snk_attention_prefill_tc_split(const void* q, long long M, const void* kpool, const void* vpool,
                                            long long num_pages, const int* block_table, int max_pages,
                                            int page_size, const int* tiles, int n_tiles, void* out, int nh, int nkv,
                                            int hd, int window, float scale, int keep, const float* slopes,
-                                           const float* sink, const void* gate, long long gate_ld,
+                                           const float* sink, const void* gate, long long gate_ld, float softcap,
                                            cudaStream_t stream) {
   if (!vpool) return SNK_ERR_SIZE;
   return at_launch(q, M, kpool, vpool, num_pages, block_table, max_pages, page_size, tiles, n_tiles, out, nh, nkv,
-                   hd, window, scale, keep, slopes, sink, gate, gate_ld, stream);
+                   hd, window, scale, keep, slopes, sink, gate, gate_ld, softcap, stream);
 }
 
 // Queue a copy of the status word into ``host`` (pinned host memory, one int) on ``stream`` without waiting

@@ -66,6 +66,16 @@ __device__ __forceinline__ float glu_out(float g, float u, int act) {
   return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
 }
 
+// The activation of an UNGATED product's store, also carried by the `swiglu` argument (the output keeps its width).
+enum { SNK_ACT_RELU2 = 5 };
+__device__ __forceinline__ float unary_out(float v, int act) {
+  if (act == SNK_ACT_RELU2) {
+    v = fmaxf(v, 0.f);
+    v *= v;
+  }
+  return v;
+}
+
 // Four consecutive outputs in the compute dtype, by one store (16-byte aligned for float, 8 for bfloat16).
 template <typename T> __device__ __forceinline__ void store4(T* p, float a, float b, float c, float d);
 template <> __device__ __forceinline__ void store4<float>(float* p, float a, float b, float c, float d) {

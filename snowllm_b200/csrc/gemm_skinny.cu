@@ -181,7 +181,7 @@ gemm_skinny_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W, OutT*
           for (int idx = threadIdx.x; idx < MT * 8 * SK_ROWS; idx += SK_WARPS * 32) {
             const int tok = idx / SK_ROWS, r = idx % SK_ROWS;
             const int m = m0 + tok, n = n0 + r;
-            if (m < row_end && n < N) C[(size_t)m * N + n] = from_f<OutT>(red[1][tok][r]);
+            if (m < row_end && n < N) C[(size_t)m * N + n] = from_f<OutT>(unary_out(red[1][tok][r], act));
           }
         }
       }
@@ -210,7 +210,7 @@ gemm_skinny_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W, OutT*
           float s = 0.f;
 #pragma unroll
           for (int w = 0; w < SK_WARPS; ++w) s += red[w][tok][r];
-          C[(size_t)m * N + n] = from_f<OutT>(s);
+          C[(size_t)m * N + n] = from_f<OutT>(unary_out(s, act));
         }
       }
     }
@@ -224,7 +224,8 @@ static int launch_skinny(const void* A, const void* W, void* C, int M, int N, in
   dim3 grid((N + SK_ROWS - 1) / SK_ROWS, offsets ? groups : 1, split);
   const dim3 block(SK_WARPS * 32);
   const bf16 *a = static_cast<const bf16*>(A), *w = static_cast<const bf16*>(W);
-  if (swiglu)
+  const int unary = swiglu == SNK_ACT_RELU2 ? swiglu : 0;
+  if (swiglu && !unary)
     snk_launch_cluster(gemm_skinny_kernel<MT, bf16, true>, grid, block, 0, stream, split, a, w,
                        static_cast<bf16*>(C), M, N, K, a_rows, a_div, offsets, swiglu);
   else if (out_f32)
@@ -232,7 +233,7 @@ static int launch_skinny(const void* A, const void* W, void* C, int M, int N, in
                        static_cast<float*>(C), M, N, K, a_rows, a_div, offsets, 0);
   else
     snk_launch_cluster(gemm_skinny_kernel<MT, bf16, false>, grid, block, 0, stream, split, a, w,
-                       static_cast<bf16*>(C), M, N, K, a_rows, a_div, offsets, 0);
+                       static_cast<bf16*>(C), M, N, K, a_rows, a_div, offsets, unary);
   SNK_LAUNCH_CHECK();
   return 0;
 }
@@ -257,13 +258,14 @@ static int skinny_split(int N, int K, const int* offsets) {
 
 // rows_hint: the most rows one group (or the whole product) is expected to hold; picks how many
 // 8-token tiles a pass covers.  More rows than that still give the right result, in more passes.
-// swiglu: W is gate/up interleaved in blocks of 8 rows and C is [M, N/2] bfloat16 = silu(gate) * up.
+// swiglu: W is gate/up interleaved in blocks of 8 rows and C is [M, N/2] bfloat16 = silu(gate) * up (or, SNK_ACT_RELU2:
+// C is [M, N] bfloat16, the square of relu of the product).
 SNK_API int snk_gemm_skinny(const void* A, const void* W, void* C, int M, int N, int K, const int* a_rows,
                             int a_div, const int* offsets, int groups, int rows_hint, int out_f32, int swiglu,
                             cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || K % 8) return SNK_ERR_SIZE;
-  if (swiglu && (N % 16 || out_f32)) return SNK_ERR_SIZE;
+  if (swiglu && ((swiglu != SNK_ACT_RELU2 && N % 16) || out_f32)) return SNK_ERR_SIZE;
   if (((uintptr_t)A % 16) || ((uintptr_t)W % 16)) return SNK_ERR_ALIGN;
   if (groups > 65535) return SNK_ERR_SIZE;
   if (a_div <= 0) a_div = 1;

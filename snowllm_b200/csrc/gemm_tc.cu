@@ -368,7 +368,7 @@ SNK_API int snk_gemm_tc(const void* A, const void* W, void* C, int M, int N, int
                         cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || K % 8) return SNK_ERR_SIZE;                   // TMA: the row pitch is a multiple of 16 bytes
-  if (swiglu && (N % 16 || out_f32)) return SNK_ERR_SIZE;
+  if (swiglu && (N % 16 || out_f32 || swiglu == SNK_ACT_RELU2)) return SNK_ERR_SIZE;
   if (((uintptr_t)A % 16) || ((uintptr_t)W % 16) || ((uintptr_t)C % 16)) return SNK_ERR_ALIGN;
   const int row_tiles = offsets ? max_row_tiles : (M + TC_BM - 1) / TC_BM;
   if (row_tiles <= 0) return SNK_ERR_SIZE;

@@ -451,7 +451,11 @@ gemm_tc2_grouped_kernel(const __grid_constant__ T2GMaps maps, const __grid_const
             OutT* dst = C + (size_t)(t.row0 + c0) * N + col0 + lane;
 #pragma unroll
             for (int j = 0; j < 32; ++j)
-              if (t.row0 + c0 + j < t.row_end) dst[(size_t)j * N] = from_f<OutT>(__uint_as_float(r[j]));
+              if (t.row0 + c0 + j < t.row_end) {
+                float v = __uint_as_float(r[j]);
+                if constexpr (sizeof(OutT) == 2) v = unary_out(v, act);
+                dst[(size_t)j * N] = from_f<OutT>(v);
+              }
           }
         }
       }
@@ -492,7 +496,9 @@ SNK_API int snk_gemm_tc2(const void* A, const void* W, void* C, int M, int N, in
                          int groups, int out_f32, int swiglu, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || K % 8) return SNK_ERR_SIZE;
-  if (swiglu && (N % 16 || out_f32)) return SNK_ERR_SIZE;
+  const int unary = swiglu == SNK_ACT_RELU2 ? swiglu : 0;  // (grouped products only)
+  if (unary) swiglu = 0;
+  if ((swiglu && N % 16) || ((swiglu || unary) && out_f32) || (unary && !offsets)) return SNK_ERR_SIZE;
   if (((uintptr_t)A % 16) || ((uintptr_t)W % 16) || ((uintptr_t)C % 16)) return SNK_ERR_ALIGN;
   if (offsets) {
     if (groups <= 0 || groups > T2G_MAX_GROUPS) return SNK_ERR_SIZE;
@@ -506,7 +512,7 @@ SNK_API int snk_gemm_tc2(const void* A, const void* W, void* C, int M, int N, in
     if (rc) return rc;
     if (swiglu) return launch_tc2_grouped<bf16, true>(maps, gw, C, M, N, K, offsets, groups, stream, swiglu);
     if (out_f32) return launch_tc2_grouped<float, false>(maps, gw, C, M, N, K, offsets, groups, stream, 0);
-    return launch_tc2_grouped<bf16, false>(maps, gw, C, M, N, K, offsets, groups, stream, 0);
+    return launch_tc2_grouped<bf16, false>(maps, gw, C, M, N, K, offsets, groups, stream, unary);
   }
   const int row_tiles = (M + 2 * T2_BM - 1) / (2 * T2_BM);
   if (row_tiles <= 0) return SNK_ERR_SIZE;

@@ -12,8 +12,10 @@
 // Every step is optional (no y: the row is only recorded and normalised).  With `rows` only those rows come out
 // and neither the residual nor the history is written (the model's last norm on the rows whose logits are wanted).
 // Sums, statistics, gates and the residual are float.  A block takes one row and keeps it in registers; its size
-// depends on W alone, so a row's sums do not depend on the batch.
+// depends on W alone and, through one threshold, on the number of rows (the order of a row's sums with it).
 #include "common.cuh"
+
+#define SW_MANY_ROWS 160       // from here on rows fill the SMs: blocks with fewer registers, more of them on an SM
 
 template <typename T> struct SwRaw;                       // four elements of the compute dtype
 template <> struct SwRaw<float> {
@@ -64,7 +66,8 @@ struct SandwichArgs {
   int W;
 };
 
-template <typename T, int VEC, int IT>
+// EARLY: for the few rows of a decode step, where a row's latency counts and not how many rows an SM holds.
+template <typename T, int VEC, int IT, bool EARLY>
 __global__ void __launch_bounds__(VEC == 4 ? 512 : 1024)
 sandwich_norm_kernel(const SandwichArgs a, T* __restrict__ out) {
   pdl_begin();
@@ -83,6 +86,48 @@ sandwich_norm_kernel(const SandwichArgs a, T* __restrict__ out) {
       for (int e = 0; e < VEC; ++e) x[it][e] = 0.f;
     }
   }
+  float old[IT][VEC];                                      // the earlier layers' share of the average
+#pragma unroll
+  for (int it = 0; it < IT; ++it)
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) old[it][e] = 0.f;
+  auto earlier_layers = [&] {
+    constexpr int JU = EARLY ? 8 : 4;                      // entries whose loads are in flight together
+#pragma unroll JU
+    for (int j = 0; j < a.n; ++j) {
+      const float w = a.avg[j];
+      const float* hx = a.history + (size_t)j * a.history_step + m * W;
+#pragma unroll
+      for (int it = 0; it < IT; ++it) {
+        const int i = threadIdx.x * VEC + it * step;
+        if (i < W) {
+          float t[VEC];
+          sw_load<float, VEC>(hx + i, t);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) old[it][e] = fmaf(w, t[e], old[it][e]);
+        }
+      }
+    }
+  };
+  // EARLY: the loads that depend on nothing go out before the sublayer's rows are looked up
+  float g[EARLY ? IT : 1][VEC], gb[EARLY ? IT : 1][VEC], w1[EARLY ? IT : 1][VEC], w2[EARLY ? IT : 1][VEC];
+  if constexpr (EARLY) {
+#pragma unroll
+    for (int it = 0; it < IT; ++it) {
+      const int i = threadIdx.x * VEC + it * step;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) g[it][e] = gb[it][e] = w1[it][e] = w2[it][e] = 0.f;
+      if (i < W) {
+        if (a.y && a.gate) {
+          sw_load<T, VEC>(static_cast<const T*>(a.gate) + m * a.gate_ld + i, g[it]);
+          sw_load<float, VEC>(a.gate_bias + i, gb[it]);
+        }
+        if (a.y && a.w1) sw_load<float, VEC>(a.w1 + i, w1[it]);
+        sw_load<float, VEC>(a.w2 + i, w2[it]);
+      }
+    }
+    if (a.avg) earlier_layers();
+  }
   if (a.y) {
     float d[IT][VEC];
     if (a.pair_pos) {
@@ -91,7 +136,7 @@ sandwich_norm_kernel(const SandwichArgs a, T* __restrict__ out) {
 #pragma unroll
         for (int e = 0; e < VEC; ++e) d[it][e] = 0.f;
       float own = 0.f;                                    // the weight of the picks that stand for h itself
-#pragma unroll 2
+#pragma unroll 4
       for (int j = 0; j < a.k; ++j) {
         const int at = a.pair_pos[m * a.k + j];
         const float w = a.pair_w[m * a.k + j];
@@ -141,12 +186,15 @@ sandwich_norm_kernel(const SandwichArgs a, T* __restrict__ out) {
 #pragma unroll
       for (int it = 0; it < IT; ++it) {
         const int i = threadIdx.x * VEC + it * step;
-        if (i < W) {
-          float g[VEC], b[VEC];
-          sw_load<T, VEC>(gr + i, g);
+        if constexpr (EARLY) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) d[it][e] /= 1.f + expf(-(g[it][e] + gb[it][e]));
+        } else if (i < W) {
+          float z[VEC], b[VEC];
+          sw_load<T, VEC>(gr + i, z);
           sw_load<float, VEC>(a.gate_bias + i, b);
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) d[it][e] /= 1.f + expf(-(g[e] + b[e]));
+          for (int e = 0; e < VEC; ++e) d[it][e] /= 1.f + expf(-(z[e] + b[e]));
         }
       }
     }
@@ -161,7 +209,10 @@ sandwich_norm_kernel(const SandwichArgs a, T* __restrict__ out) {
 #pragma unroll
       for (int it = 0; it < IT; ++it) {
         const int i = threadIdx.x * VEC + it * step;
-        if (i < W) {
+        if constexpr (EARLY) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) x[it][e] = fmaf(d[it][e] * inv, w1[it][e], x[it][e]);
+        } else if (i < W) {
           float w[VEC];
           sw_load<float, VEC>(a.w1 + i, w);
 #pragma unroll
@@ -184,26 +235,12 @@ sandwich_norm_kernel(const SandwichArgs a, T* __restrict__ out) {
     }
   }
   if (a.avg) {
+    if constexpr (!EARLY) earlier_layers();
     const float last = a.avg[a.n];
 #pragma unroll
     for (int it = 0; it < IT; ++it)
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) x[it][e] *= last;
-#pragma unroll 4
-    for (int j = 0; j < a.n; ++j) {
-      const float w = a.avg[j];
-      const float* hx = a.history + (size_t)j * a.history_step + m * W;
-#pragma unroll
-      for (int it = 0; it < IT; ++it) {
-        const int i = threadIdx.x * VEC + it * step;
-        if (i < W) {
-          float t[VEC];
-          sw_load<float, VEC>(hx + i, t);
-#pragma unroll
-          for (int e = 0; e < VEC; ++e) x[it][e] = fmaf(w, t[e], x[it][e]);
-        }
-      }
-    }
+      for (int e = 0; e < VEC; ++e) x[it][e] = fmaf(last, x[it][e], old[it][e]);
   }
   float ss = 0.f;
 #pragma unroll
@@ -222,9 +259,9 @@ sandwich_norm_kernel(const SandwichArgs a, T* __restrict__ out) {
     const int i = threadIdx.x * VEC + it * step;
     if (i < W) {
       float w[VEC], o[VEC];
-      sw_load<float, VEC>(a.w2 + i, w);
+      if constexpr (!EARLY) sw_load<float, VEC>(a.w2 + i, w);
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) o[e] = x[it][e] * inv * w[e];
+      for (int e = 0; e < VEC; ++e) o[e] = x[it][e] * inv * (EARLY ? w2[it][e] : w[e]);
       sw_store<T, VEC>(out + (size_t)blockIdx.x * W + i, o);
     }
   }
@@ -245,12 +282,18 @@ SNK_API int snk_sandwich_norm(float* residual, const float* y, const int* pair_p
                    ((uintptr_t)residual | (uintptr_t)y | (uintptr_t)gate_bias | (uintptr_t)w1 | (uintptr_t)history |
                     (uintptr_t)w2) % 16 == 0 &&
                    ((uintptr_t)h | (uintptr_t)gate | (uintptr_t)out) % tv == 0;
-#define SW_LAUNCH(VEC_, IT_, THREADS_)                                                                        \
-  snk_launch(sandwich_norm_kernel<T, VEC_, IT_>, dim3(R), dim3(THREADS_), 0, stream, args, static_cast<T*>(out))
+#define SW_LAUNCH_(VEC_, IT_, EARLY_, THREADS_)                                                               \
+  snk_launch(sandwich_norm_kernel<T, VEC_, IT_, EARLY_>, dim3(R), dim3(THREADS_), 0, stream, args, static_cast<T*>(out))
+#define SW_LAUNCH(VEC_, IT_, THREADS_) SW_LAUNCH_(VEC_, IT_, false, THREADS_)
   SNK_DISPATCH(dtype, {
     if (vec) {
       const int n4 = W / 4;
-      if (n4 <= 64) SW_LAUNCH(4, 1, 64);
+      if (R < SW_MANY_ROWS && n4 <= 1024) {
+        if (n4 <= 64) SW_LAUNCH_(4, 1, true, 64);
+        else if (n4 <= 256) SW_LAUNCH_(4, 1, true, 256);
+        else if (n4 <= 512) SW_LAUNCH_(4, 1, true, 512);
+        else SW_LAUNCH_(4, 2, true, 512);
+      } else if (n4 <= 64) SW_LAUNCH(4, 1, 64);
       else if (n4 <= 256) SW_LAUNCH(4, 1, 256);
       else if (n4 <= 512) SW_LAUNCH(4, 2, 256);
       else if (n4 <= 1024) SW_LAUNCH(4, 4, 256);
@@ -264,6 +307,7 @@ SNK_API int snk_sandwich_norm(float* residual, const float* y, const int* pair_p
     }
   });
 #undef SW_LAUNCH
+#undef SW_LAUNCH_
   SNK_LAUNCH_CHECK();
   return 0;
 }

@@ -295,11 +295,14 @@ SNK_API int snk_short_conv(const void* bcx, const void* w, int w_is_f32, void* s
 // history holds the same values that a longer step would read from its own rows: a sequence gives the
 // same bits however it is cut.  Launches as above: one that only reads the state and one that rewrites
 // it; steps of one token per segment do both in one.
-__device__ __forceinline__ float conv_silu(float z) { return z / (1.f + expf(-z)); }
+template <typename T> __device__ __forceinline__ float conv_silu(float z) { return z / (1.f + expf(-z)); }
+// rounded to bfloat16 at the store: the special-function unit's exponential and reciprocal are exact enough
+template <> __device__ __forceinline__ float conv_silu<bf16>(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 // The taps' sum with the channel's bias (where there is one) and the activation.
+template <typename T>
 __device__ __forceinline__ float conv_end(float acc, const SmallVec& cb, int c, int silu) {
   const float z = acc + (cb.p ? cb[c] : 0.f);
-  return silu ? conv_silu(z) : z;
+  return silu ? conv_silu<T>(z) : z;
 }
 
 template <typename T>
@@ -325,7 +328,7 @@ __global__ void causal_conv_kernel(const T* __restrict__ u, long long ld, SmallV
     else v = has_state ? to_f<T>(st[(size_t)(s + L - 1) * C + c]) : 0.f;
     acc = fmaf(w[(size_t)c * L + j], v, acc);
   }
-  out[(size_t)m * out_ld + c] = from_f<T>(conv_end(acc, cb, c, silu));
+  out[(size_t)m * out_ld + c] = from_f<T>(conv_end<T>(acc, cb, c, silu));
 }
 
 template <typename T>
@@ -376,10 +379,58 @@ __global__ void causal_conv_decode_kernel(const T* __restrict__ u, long long ld,
   for (int j = 0; j < CONV_MAX_L; ++j)
     if (j < L - 1) acc = fmaf(w[(size_t)c * L + j], to_f<T>(hist[j]), acc);
   acc = fmaf(w[(size_t)c * L + L - 1], to_f<T>(cur), acc);
-  out[(size_t)seg * out_ld + c] = from_f<T>(conv_end(acc, cb, c, silu));
+  out[(size_t)seg * out_ld + c] = from_f<T>(conv_end<T>(acc, cb, c, silu));
 #pragma unroll
   for (int j = 0; j < CONV_MAX_L; ++j)
     if (j < L - 1) st[(size_t)j * C + c] = j + 1 < L - 1 ? hist[j + 1] : cur;
+}
+
+// One token per segment, four consecutive channels a thread (8- or 16-byte accesses): every load of the history, the
+// row and the taps is issued before the first is used.  Taps in order, as the kernels above.
+template <typename T, int L>
+__global__ void __launch_bounds__(128)
+causal_conv_decode_vec_kernel(const T* __restrict__ u, long long ld, SmallVec w, T* __restrict__ state,
+                              const int* __restrict__ seg_start, const int* __restrict__ seg_slot,
+                              T* __restrict__ out, long long out_ld, int C, SmallVec cb, int silu) {
+  pdl_begin();
+  constexpr int VEC = ConvVec<T>::N;
+  using Raw = typename ConvVec<T>::Raw;
+  const int c0 = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+  if (c0 >= C) return;
+  const int seg = blockIdx.y;                        // = the row
+  T* st = state + (size_t)seg_slot[seg] * (L - 1) * C + c0;
+  const bool has_state = seg_start[seg] > 0;
+  Raw raw[L];                                        // history, then the current token
+  raw[L - 1] = *reinterpret_cast<const Raw*>(u + (size_t)seg * ld + c0);
+#pragma unroll
+  for (int j = 0; j < L - 1; ++j) raw[j] = *reinterpret_cast<const Raw*>(st + (size_t)j * C);
+  float acc[VEC], bias[VEC], taps[VEC][L];
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) {
+    bias[e] = cb.p ? cb[c0 + e] : 0.f;
+    acc[e] = 0.f;
+#pragma unroll
+    for (int j = 0; j < L; ++j) taps[e][j] = w[(size_t)(c0 + e) * L + j];
+  }
+  Raw none;
+  {
+    const float zero[VEC] = {};
+    none = ConvVec<T>::pack(zero);
+  }
+#pragma unroll
+  for (int j = 0; j < L; ++j) {
+    if (j < L - 1 && !has_state) raw[j] = none;      // a fresh request: whatever the slot holds is not its own
+    float v[VEC];
+    ConvVec<T>::unpack(raw[j], v);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) acc[e] = fmaf(taps[e][j], v[e], acc[e]);
+  }
+  float y[VEC];
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) y[e] = silu ? conv_silu<T>(acc[e] + bias[e]) : acc[e] + bias[e];
+  *reinterpret_cast<Raw*>(out + (size_t)seg * out_ld + c0) = ConvVec<T>::pack(y);
+#pragma unroll
+  for (int j = 0; j < L - 1; ++j) *reinterpret_cast<Raw*>(st + (size_t)j * C) = raw[j + 1];
 }
 
 // Many rows (prompt portions): as short_conv_strip_kernel above, without the gates.  A thread owns four
@@ -452,7 +503,7 @@ causal_conv_strip_kernel(const T* __restrict__ u, long long ld, SmallVec w, cons
 #pragma unroll
         for (int i = 0; i < L - 1; ++i) acc = fmaf(taps[i][e], hist[i][e], acc);
         acc = fmaf(taps[L - 1][e], x[e], acc);
-        y[e] = silu ? conv_silu(acc + bias[e]) : acc + bias[e];
+        y[e] = silu ? conv_silu<T>(acc + bias[e]) : acc + bias[e];
 #pragma unroll
         for (int i = 0; i < L - 2; ++i) hist[i][e] = hist[i + 1][e];
         if (L > 1) hist[L - 2 < 0 ? 0 : L - 2][e] = x[e];
@@ -471,6 +522,25 @@ SNK_API int snk_causal_conv(const void* u, long long ld, const void* w, int w_is
   if (L < 1 || L > CONV_MAX_L || M > 65535 * 64 || B > 65535) return SNK_ERR_SIZE;
   const int threads = 128;
   SmallVec wv{w, w_is_f32}, cb{bias, w_is_f32};
+  const size_t vbytes = dtype == SNK_F32 ? 16 : 8;   // four channels per thread
+  const size_t esz = dtype == SNK_F32 ? 4 : 2;
+  const bool aligned = C % 4 == 0 && (uintptr_t)u % vbytes == 0 && (uintptr_t)state % vbytes == 0 &&
+                       (uintptr_t)out % vbytes == 0 && (ld * esz) % vbytes == 0 && (out_ld * esz) % vbytes == 0;
+  if (M == B && L >= 2 && L <= CONV_FAST_L && aligned) {
+    dim3 vgrid((C / 4 + threads - 1) / threads, B);
+#define CAUSAL_DECODE_LAUNCH(L_)                                                                         \
+    snk_launch(causal_conv_decode_vec_kernel<T, L_>, dim3(vgrid), dim3(threads), 0, stream,              \
+               static_cast<const T*>(u), ld, wv, static_cast<T*>(state), seg_start, seg_slot,            \
+               static_cast<T*>(out), out_ld, C, cb, silu)
+    SNK_DISPATCH(dtype, {
+      if (L == 2) CAUSAL_DECODE_LAUNCH(2);
+      else if (L == 3) CAUSAL_DECODE_LAUNCH(3);
+      else CAUSAL_DECODE_LAUNCH(4);
+    });
+#undef CAUSAL_DECODE_LAUNCH
+    SNK_LAUNCH_CHECK();
+    return 0;
+  }
   if (M == B && L > 1) {                             // one token per segment
     dim3 dgrid((C + threads - 1) / threads, B);
     SNK_DISPATCH(dtype, snk_launch(causal_conv_decode_kernel<T>, dim3(dgrid), dim3(threads), 0, stream,
@@ -479,10 +549,6 @@ SNK_API int snk_causal_conv(const void* u, long long ld, const void* w, int w_is
     SNK_LAUNCH_CHECK();
     return 0;
   }
-  const size_t vbytes = dtype == SNK_F32 ? 16 : 8;   // four channels per thread
-  const size_t esz = dtype == SNK_F32 ? 4 : 2;
-  const bool aligned = C % 4 == 0 && (uintptr_t)u % vbytes == 0 && (uintptr_t)state % vbytes == 0 &&
-                       (uintptr_t)out % vbytes == 0 && (ld * esz) % vbytes == 0 && (out_ld * esz) % vbytes == 0;
   if (L >= 2 && L <= CONV_FAST_L && aligned && M >= 4 * CONV_STRIP) {
     dim3 sgrid((C / 4 + threads - 1) / threads, (M + CONV_STRIP - 1) / CONV_STRIP);
     if (sgrid.y > 65535u) return SNK_ERR_SIZE;

@@ -93,6 +93,8 @@ class Model:
     def finish_binding(self) -> None:
         if getattr(self.head, "tied", False):
             self.head.bind({"weight": self.embedding.weight})
+        for block in self.blocks:              # an arrangement may join weights of several of its parts
+            getattr(block, "finish_binding", lambda: None)()
         self.bound = True
 
     EMBEDDING_CACHE = "embedding"      # the key of an embedding's own state among the cache specs

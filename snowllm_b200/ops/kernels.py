@@ -47,13 +47,13 @@ _SIGNATURES = {
         "snk_attention_decode_mma": [P, P, P, I, I, P, P, P, P, P, I, I, I, I, I, I, F, P],
         "snk_attention_prefill_tma": [P, P, LL, P, I, I, P, I, P, I, I, I, I, F, P],
         "snk_attention_decode_tma": [P, P, LL, P, I, I, P, P, P, P, P, I, I, I, I, I, I, F, P],
-        "snk_attention_decode_tma_split": [P, P, P, LL, P, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, P, P, P, LL, P],
+        "snk_attention_decode_tma_split": [P, P, P, LL, P, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, P, P, P, LL, F, P],
         "snk_attention_decode_status": [],
         "snk_attention_decode_status_peek": [P, P],
     },
     "attention_tc": {
         "snk_attention_prefill_tc": [P, LL, P, LL, P, I, I, P, I, P, I, I, I, I, F, P],
-        "snk_attention_prefill_tc_split": [P, LL, P, P, LL, P, I, I, P, I, P, I, I, I, I, F, I, P, P, P, LL, P],
+        "snk_attention_prefill_tc_split": [P, LL, P, P, LL, P, I, I, P, I, P, I, I, I, I, F, I, P, P, P, LL, F, P],
         "snk_attention_tc_status": [],
         "snk_attention_tc_status_peek": [P, P],
     },
@@ -629,10 +629,10 @@ def attention_prefill_tc(q, pool, block_table, page_size, tiles, scale, out, win
 
 
 def attention_prefill_tc_split(q, kpool, vpool, block_table, page_size, tiles, scale, out, *, window=None, keep=0,
-                               slopes=None, sink=None, gate=None, gate_col=0):
+                               slopes=None, sink=None, gate=None, gate_col=0, softcap=None):
     """``attention_prefill_tc`` over keys and values in pools of their own [pages, kv heads, page_size, 64], with
     the options of ``split_attention``: ``keep`` first positions beside the window, ``slopes`` and ``sink`` float
-    [heads], ``gate`` [M, width] bfloat16 whose columns from ``gate_col`` hold a logit per head."""
+    [heads], ``gate`` [M, width] bfloat16 whose columns from ``gate_col`` hold a logit per head, ``softcap``."""
     M, nh, hd = q.shape
     _chk(q, "q", torch.bfloat16)
     _chk(kpool, "key pool", torch.bfloat16)
@@ -669,7 +669,7 @@ def attention_prefill_tc_split(q, kpool, vpool, block_table, page_size, tiles, s
     check(fn("snk_attention_prefill_tc_split")(
         _ptr(q), M, _ptr(kpool), _ptr(vpool), kpool.shape[0], _ptr(block_table), block_table.shape[1], page_size,
         _ptr(tiles), tiles.shape[0], _ptr(out), nh, nkv, hd, int(window or 0), float(scale), int(keep or 0),
-        _ptr(slopes), _ptr(sink), gate_ptr, gate_ld, _stream()), "attention_prefill_tc", work=work)
+        _ptr(slopes), _ptr(sink), gate_ptr, gate_ld, float(softcap or 0.0), _stream()), "attention_prefill_tc", work=work)
     return out
 
 
@@ -749,12 +749,12 @@ def attention_decode_mma(q, pool, block_table, page_size, positions, row_seg, sc
 
 def attention_decode_tma_split(q, kpool, vpool, block_table, page_size, positions, row_seg, scale, num_chunks, out, *,
                                window=None, keep=0, slopes=None, sink=None, gate=None, gate_col=0, scratch=None,
-                               rows=None):
+                               rows=None, softcap=None):
     """``attention_decode_mma`` by TMA over keys and values in pools of their own [pages, kv heads, page_size,
     64 or 128], with the options of ``split_attention``: ``keep`` first positions beside the window (a row's
     chunks of 256 keys are then the chunks of its kept keys followed by its window's; ``num_chunks`` counts
     both), ``slopes`` and ``sink`` float [heads], ``gate`` [M, width] bfloat16 whose columns from ``gate_col``
-    hold a logit per head.  Every served row stands alone; ``rows`` (int32, on the device): the rows of the
+    hold a logit per head, ``softcap``.  Every served row stands alone; ``rows`` (int32, on the device): the rows of the
     step to serve, when not all of them (the others' outputs are left as they are)."""
     M, nh, hd = q.shape
     served = M
@@ -803,7 +803,7 @@ def attention_decode_tma_split(q, kpool, vpool, block_table, page_size, position
     check(fn("snk_attention_decode_tma_split")(
         _ptr(q), _ptr(kpool), _ptr(vpool), kpool.shape[0], _ptr(block_table), block_table.shape[1], page_size,
         _ptr(positions), _ptr(row_seg), _ptr(rows), _ptr(out), _ptr(scratch), served, nh, nkv, hd, int(window or 0),
-        num_chunks, float(scale), keep, _ptr(slopes), _ptr(sink), gate_ptr, gate_ld, _stream()),
+        num_chunks, float(scale), keep, _ptr(slopes), _ptr(sink), gate_ptr, gate_ld, float(softcap or 0.0), _stream()),
         "attention_decode_tma", work=work)
     if num_chunks > 1:
         check(fn("snk_attention_merge_gated")(_ptr(scratch), _ptr(positions), _ptr(out), served, nh, hd,
@@ -971,9 +971,10 @@ def gemm_skinny_ok(a, w) -> bool:
 
 
 def gemm_skinny(a, w, out_dtype=None, out=None, a_rows=None, a_div=1, offsets=None, rows_out=None,
-                rows_hint=None, swiglu=False):
+                rows_hint=None, swiglu=False, act: int = 0):
     """bfloat16 a [M, K] times w [N, K]^T (or grouped w [G, N, K]) for few rows: W streams from memory
-    once into tensor-core fragments.  ``rows_hint``: rows expected per group (sets the pass size)."""
+    once into tensor-core fragments.  ``rows_hint``: rows expected per group (sets the pass size).  ``act``: the code of
+    an activation applied at the store (``UNARY_CODES``; bfloat16 output)."""
     _chk(a, "gemm a", torch.bfloat16)
     _chk(w, "gemm w", torch.bfloat16)
     K = a.shape[1]
@@ -998,11 +999,12 @@ def gemm_skinny(a, w, out_dtype=None, out=None, a_rows=None, a_div=1, offsets=No
         raise KernelError("gemm output is bfloat16 or float32 (bfloat16 with swiglu)")
     check(fn("snk_gemm_skinny")(_ptr(a), _ptr(w), _ptr(out), M, N, K, _ptr(a_rows), int(a_div), _ptr(offsets),
                                 G, int(rows_hint if rows_hint is not None else M),
-                                int(out_dtype == torch.float32), int(swiglu), _stream()), "gemm_skinny",
+                                int(out_dtype == torch.float32), int(swiglu or act), _stream()), "gemm_skinny",
           work=lambda: _gemm_work(M, a, w, out, offsets))
     return out
 
 
+UNARY_CODES = {"relu2": 5}       # activations that an ungated product's store can apply
 TC_TILE = 128
 
 
@@ -1044,11 +1046,12 @@ def gemm_tc(a, w, out_dtype=None, out=None, offsets=None, swiglu=False):
     return out
 
 
-def gemm_tc2(a, w, out_dtype=None, out=None, offsets=None, swiglu=False):
+def gemm_tc2(a, w, out_dtype=None, out=None, offsets=None, swiglu=False, act: int = 0):
     """As ``gemm_tc``, on pairs of SMs (cta_group::2): 256 x 256 tiles of C, each block of a pair loading
     its 128 rows of ``a`` and half of the tile's rows of ``w``.  Grouped (``offsets``): the operands change
     places, each block loads 128 rows of the group's ``w`` and half of up to 256 of its rows of ``a``, and
-    a group's last tile is as wide as its rows need (a multiple of 16); at most 256 groups."""
+    a group's last tile is as wide as its rows need (a multiple of 16); at most 256 groups.  ``act`` (grouped, bfloat16
+    output): the code of an activation applied at the store (``UNARY_CODES``)."""
     _chk(a, "gemm a", torch.bfloat16)
     _chk(w, "gemm w", torch.bfloat16)
     M, K = a.shape
@@ -1069,7 +1072,7 @@ def gemm_tc2(a, w, out_dtype=None, out=None, offsets=None, swiglu=False):
     if out_dtype not in (torch.bfloat16, torch.float32) or (swiglu and out_dtype != torch.bfloat16):
         raise KernelError("gemm output is bfloat16 or float32 (bfloat16 with swiglu)")
     check(fn("snk_gemm_tc2")(_ptr(a), _ptr(w), _ptr(out), M, N, K, _ptr(offsets), G,
-                             int(out_dtype == torch.float32), int(swiglu), _stream()), "gemm_tc2",
+                             int(out_dtype == torch.float32), int(swiglu or act), _stream()), "gemm_tc2",
           work=lambda: _gemm_work(M, a, w, out, offsets))
     return out
 

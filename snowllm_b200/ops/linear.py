@@ -71,6 +71,20 @@ def grouped_linear(x, w, offsets, rows_out, max_rows_per_group, a_rows=None, a_d
                              rows_out=rows_out, max_rows_per_group=max_rows_per_group)
 
 
+def grouped_linear_act(x, w, offsets, rows_out, max_rows_per_group, a_rows, a_div, activation: str):
+    """The grouped product with ``activation`` on its output (ungated experts); the bfloat16 products apply the square
+    of relu at their store, otherwise one elementwise kernel follows."""
+    code = kernels.UNARY_CODES.get(activation)
+    if code is not None and kernels.gemm_skinny_ok(x, w) and w.shape[0] <= PAIRS_MAX_GROUPS and TC_PAIRS:
+        if _few_rows_per_group(rows_out, w.shape[0]):
+            hint = min(max_rows_per_group, max(8, 2 * -(-rows_out // w.shape[0])))
+            return kernels.gemm_skinny(x, w, a_rows=a_rows, a_div=a_div, offsets=offsets, rows_out=rows_out,
+                                       rows_hint=hint, act=code)
+        xs = kernels.gather_rows(x, a_rows, a_div) if a_rows is not None else x
+        return kernels.gemm_tc2(xs, w, offsets=offsets, act=code)
+    return kernels.act_rows(grouped_linear(x, w, offsets, rows_out, max_rows_per_group, a_rows, a_div), activation)
+
+
 def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
     """[..., I, K] gate and up rows -> [..., 2I, K] in blocks of 8 gate rows followed by the 8 up rows of
     the same features: the layout whose product can apply SwiGLU at its store (I a multiple of 8)."""

@@ -123,6 +123,7 @@ class MapsAttention(Part):
     norm_weights = True        # the per-head norm of q and k has a weight (False: the plain root mean square)
     whole_norm = False         # True: ONE root mean square over all heads of q (of k), weights of that size
     keep_first = 0             # positions at the sequence's start that stay reachable beside the window
+    _lends_rows = False        # whether the fused projection carries rows of another part (``append_input_rows``)
     softcap = None             # c: a scaled score s becomes c * tanh(s / c)
 
     def __init__(self, dtype, names, *, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int,
@@ -206,12 +207,26 @@ class MapsAttention(Part):
         self.q_norm = tensors.get("q_norm")
         self.k_norm = tensors.get("k_norm", self.q_norm)      # a reader of another layer's cache normalises q alone
 
+    def append_input_rows(self, weight) -> int:
+        """Further rows for the fused projection (``Part``): the column their outputs start at."""
+        col = self.w_in.shape[0]
+        self.w_in = pad_rows(torch.cat((self.w_in, weight), 0), 16)
+        if self.proj_bias is not None:
+            self.proj_bias = torch.cat((self.proj_bias, self.proj_bias.new_zeros(self.w_in.shape[0] - col))).contiguous()
+        self._lends_rows = True
+        return col
+
+    def input_rows(self, ctx):
+        return ctx.memo.pop(("input_rows", id(self)))
+
     # -- the step -----------------------------------------------------------------------------
     def _attend(self, ctx, x, cache, owns_cache, out_dtype):
         if owns_cache == self.reads_cache:
             raise KernelError("a layer without key and value tensors must read another layer's cache, "
                               "and one with them must own its cache")
         proj = linear(x, self.w_in)
+        if self._lends_rows:
+            ctx.memo[("input_rows", id(self))] = proj
         q_off, k_off, v_off, g_off, _ = self._columns()
         cache, rows = self._convolved(ctx, proj, cache)      # the rows that are normalised, turned and cached
         kpool, vpool = cache.pools
@@ -231,7 +246,7 @@ class MapsAttention(Part):
             kernels.attention_prefill_tc_split(q, kpool, vpool, cache.block_table, cache.page_size, tc_tiles, self.scale,
                                                out, window=self.window, keep=self.keep_first, slopes=self.slopes,
                                                sink=self.sink, gate=proj if self._gate_in_kernel() else None,
-                                               gate_col=g_off)
+                                               gate_col=g_off, softcap=self.softcap)
             if not rows_host:
                 ctx.tap("attention_o", out)
                 return proj, out
@@ -249,15 +264,15 @@ class MapsAttention(Part):
         keys and values alike, a mask and a bias it knows (causal, a window with or without kept first keys, a
         slope per head, a sink per head, a gate per head)."""
         return (self.maps == 1 and self.head_dim == 64 and self.v_head_dim == 64 and self.bias is None
-                and self.block is None and self.head_scale is None and self.softcap is None
-                and out_dtype == torch.bfloat16 and kernels.attention_prefill_tc_ok(q, cache.page_size)
+                and self.block is None and self.head_scale is None and out_dtype == torch.bfloat16
+                and kernels.attention_prefill_tc_ok(q, cache.page_size)
                 and max(ctx.host_seg_len) >= plan.PREFILL_MIN_ROWS)
 
     def _decode_kernel_ok(self, q, cache, out_dtype) -> bool:
         """Whether rows that stand alone go to the TMA decode kernel: bfloat16, one map, heads of 64 or 128 for
         keys and values alike, up to 16 heads per kv head, a mask and a bias it knows."""
         return (self.maps == 1 and self.head_dim == self.v_head_dim and self.head_dim in kernels.PREFILL_HEAD_DIMS
-                and self.bias is None and self.block is None and self.head_scale is None and self.softcap is None
+                and self.bias is None and self.block is None and self.head_scale is None
                 and out_dtype == torch.bfloat16 and q.dtype == torch.bfloat16
                 and self.nq // self.num_kv_heads <= kernels.DECODE_MMA_MAX_GROUP
                 and kernels.DECODE_TMA and kernels.decode_tma_page_ok(cache.page_size))
@@ -277,7 +292,7 @@ class MapsAttention(Part):
                                            ctx.row_seg, self.scale, num_chunks, out, window=self.window,
                                            keep=self.keep_first, slopes=self.slopes, sink=self.sink,
                                            gate=proj if self._gate_in_kernel() else None, gate_col=g_off,
-                                           scratch=scratch, rows=rows_dev)
+                                           scratch=scratch, rows=rows_dev, softcap=self.softcap)
 
     def _rows(self, ctx, q, cache, proj, g_off, out_dtype, tiles, tile_rows, out):
         """The kernels of csrc/attention_split.cu: every row of the step (``tiles`` None), or the rows that

@@ -45,6 +45,11 @@ class Part:
     def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
         """Take the loaded tensors (keyed by TensorSpec.local), fuse or reshape as needed."""
 
+    # A part whose first product reads its input as it is may take further rows into that product:
+    # ``append_input_rows(weight [n, hidden]) -> first column`` after ``bind``, and ``input_rows(ctx) -> [M, width]``,
+    # the product's output, after ``forward`` of a step (an output gate on the same input then costs no product of its
+    # own).  Parts that do not offer it have no such methods.
+
     def parts(self):
         """Parts nested in this one (a mixer made of two mixers): the model declares and binds their tensors as
         it does this part's own."""

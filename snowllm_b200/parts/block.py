@@ -263,13 +263,14 @@ class HyperBlock:
 
 class OutputGate(Part):
     """A gate per element on a sublayer's output, sigmoid(W h + b) of the sublayer's input h: the logits W h come from
-    one product in the compute dtype, bias and sigmoid are applied in float by the norm that adds the output."""
+    a product in the compute dtype (the sublayer's own first one, where it takes further rows), bias and sigmoid are
+    applied in float by the norm that adds the output."""
     libraries = ("gemm", "gemm_skinny", "gemm_tc", "gemm_tc2")
 
     def __init__(self, dtype, names, *, hidden_size: int):
         super().__init__(dtype, names)
         self.hidden_size = hidden_size
-        self.weight = self.bias = None
+        self.weight = self.bias = self._rides = None
 
     def declare(self, has):
         W, n = self.hidden_size, self.names
@@ -278,8 +279,17 @@ class OutputGate(Part):
     def bind(self, tensors):
         self.weight, self.bias = tensors["weight"], tensors["bias"]
 
+    def ride_in(self, sublayer) -> None:
+        """Let the sublayer's own first product form the logits, where it offers that."""
+        if hasattr(sublayer, "append_input_rows"):
+            self._rides = (sublayer, sublayer.append_input_rows(self.weight))
+            self.weight = None
+
     def forward(self, ctx, h):
         """What a ``kernels.NormedDelta`` takes as its gate."""
+        if self._rides is not None:
+            sublayer, col = self._rides
+            return sublayer.input_rows(ctx), col, self.bias
         return linear(h, self.weight), 0, self.bias
 
 
@@ -328,6 +338,11 @@ class SandwichBlock:
     def parts(self):
         own = tuple(p for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn) if p is not None)
         return own + tuple(self.post) + tuple(self.gates or ()) + ((self.average,) if self.average else ())
+
+    def finish_binding(self):
+        """Once the weights of all parts are there: a gate reads what its sublayer reads."""
+        for gate, sublayer in zip(self.gates or (), (self.mixer, self.ffn)):
+            gate.ride_in(sublayer)
 
     def _pending(self, ctx, q: int, y, h, last: bool, history):
         gate = self.gates[q].forward(ctx, h) if self.gates is not None else None

@@ -23,7 +23,7 @@ from __future__ import annotations
 import torch
 
 from ..errors import ConfigError
-from ..ops import grouped_linear, grouped_linear_glu, interleave_gate_up, kernels, linear, linear_glu
+from ..ops import grouped_linear, grouped_linear_act, grouped_linear_glu, interleave_gate_up, kernels, linear, linear_glu
 from .base import Part
 from .registry import register_ffn
 from .spec import INIT_BIAS, KEEP_F32, KEEP_SMALL, TensorSpec
@@ -188,7 +188,7 @@ class SigmoidMoE(Part):
         if not self.gated:
             # the pairs of identity experts sort behind the others and own no rows in the products
             own = offsets[:self.num_experts + 1]
-            act = kernels.act_rows(grouped_linear(x, self.w1, own, M * k, cap, sorted_pair, k), self.activation)
+            act = grouped_linear_act(x, self.w1, own, M * k, cap, sorted_pair, k, self.activation)
             y = grouped_linear(act, self.w2, own, M * k, cap, out_dtype=torch.float32)
             return kernels.ExpertSum(y, pair_pos, weights, x=x if self.identity else None)
         if self.scale_input:

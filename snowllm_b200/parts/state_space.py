@@ -27,6 +27,7 @@ MAX_CONV_TAPS = 16
 
 class Mamba2(Part):
     libraries = ("gemm", "gemm_skinny", "gemm_tc", "gemm_tc2", "short_conv", "state_space")
+    _lends_rows = False        # whether the projection carries rows of another part (``append_input_rows``)
 
     def __init__(self, dtype, names, *, hidden_size: int, num_heads: int, head_dim: int, state_size: int,
                  num_groups: int = 1, norm_groups: int = 1, conv_taps: int = 4, norm_eps: float):
@@ -84,8 +85,20 @@ class Mamba2(Part):
         self.dt_bias, self.skip = tensors["dt_bias"].contiguous(), tensors["skip"].contiguous()
         self.rate = (-torch.exp(tensors["a_log"].float())).contiguous()
 
+    def append_input_rows(self, weight) -> int:
+        """Further rows for the projection (``Part``): the column their outputs start at."""
+        col = self.w_in.shape[0]
+        self.w_in = pad_rows(torch.cat((self.w_in, weight), 0), 16)
+        self._lends_rows = True
+        return col
+
+    def input_rows(self, ctx):
+        return ctx.memo.pop(("input_rows", id(self)))
+
     def forward(self, ctx, x, cache, owns_cache=True):
         proj = linear(x, self.w_in)
+        if self._lends_rows:
+            ctx.memo[("input_rows", id(self))] = proj
         z_col, dt_col = self._columns()
         state = cache.tensors[0]
         history = cache.tensors[1] if self.conv_taps > 1 else proj.new_empty(1, 0, self.conv_channels)

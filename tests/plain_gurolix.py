@@ -80,7 +80,8 @@ def attention(h, t, m: dict, eps: float, p: str, positions, v_first=None, normed
     own = (h @ t[p + "v"].T + t[p + "v.b"]).view(T, G, dv)
     if normed:
         q, k = over_rms(q, eps) * t[p + "q.norm"], over_rms(k, eps) * t[p + "k.norm"]
-    freqs = frequencies(m["rot"]["base"], m["rot"]["dims"], m["rot"].get("scaling"))
+    rot = m.get("rot")
+    freqs = [] if rot is None else frequencies(rot["base"], rot["dims"], rot.get("scaling"))
     q, k = rotate_halves(q, positions, freqs), rotate_halves(k, positions, freqs)
     v = own
     if v_first is not None:
@@ -133,7 +134,7 @@ def mamba2(h, t, m: dict, eps: float, p: str):
     """Projection [z | x | B | C | dt]; x, B, C through a short convolution and silu; the recurrence; the gate
     silu(z) BEFORE an RMS norm in ``norm_groups`` equal parts; output product."""
     T = h.shape[0]
-    H, P, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
+    H, P, N, G = m["heads"], m["vdim"], m["state"], m.get("groups", 1)
     inner = H * P
     z, x, B, C, dt = torch.split(h @ t[p + "in"].T, [inner, inner, G * N, G * N, H], -1)
     u = silu(causal_taps(torch.cat((x, B, C), -1), t[p + "conv"], t[p + "conv.b"]))
@@ -143,7 +144,7 @@ def mamba2(h, t, m: dict, eps: float, p: str):
     decay = torch.exp(-torch.exp(t[p + "A_log"]) * step)
     y = state_space(x.view(T, H, P), B, C, step, decay, t[p + "D"]).reshape(T, inner)
     y = y * silu(z)
-    parts = m["norm_groups"]
+    parts = m.get("norm_groups", 1)
     y = over_rms(y.view(T, parts, inner // parts), eps).reshape(T, inner) * t[p + "norm"]
     return y @ t[p + "o"].T
 
@@ -165,7 +166,7 @@ def choose(choice, top: int, count: int, keep: int):
 def experts(h, t, mlp: dict, p: str, picks=None, router_input=None):
     """Scores s: the softmax over all router outputs.  s + correction chooses, s weighs (not renormalised).  An
     expert is down(relu(up h)^2); the last ``identity`` router outputs stand for the input itself.
-    ``picks`` [T, top] forces the choice."""
+    ``picks`` [T, top] forces the choice.  Returns (output, the choice)."""
     r = mlp["router"]
     E, same, g = r["experts"], r.get("identity") or 0, r.get("groups") or {"count": 1, "keep": 1}
     s = torch.softmax((h if router_input is None else router_input) @ t[p + "router"].T, -1)
@@ -182,14 +183,14 @@ def experts(h, t, mlp: dict, p: str, picks=None, router_input=None):
         else:
             y = rows
         out[hit] = out[hit] + s[hit, e:e + 1] * y
-    return out
+    return out, picks
 
 
 # --- the model ------------------------------------------------------------------------------------
 
-def forward(model: dict, tokens, dtype=torch.float64, layers_out=None, picks=None):
+def forward(model: dict, tokens, dtype=torch.float64, layers_out=None, picks=None, picks_out=None):
     """Logits [T, vocab] of one whole sequence.  ``layers_out`` (a list) receives the stream as each layer hands
-    it on; ``picks`` {layer: [T, top]} forces the experts."""
+    it on; ``picks`` {layer: [T, top]} forces the experts, ``picks_out`` (a dict) receives {layer: the choice made}."""
     cfg = model["config"]
     t = {k: v.to(dtype) for k, v in model["tensors"].items()}
     eps = cfg["norm"]["eps"]
@@ -213,7 +214,9 @@ def forward(model: dict, tokens, dtype=torch.float64, layers_out=None, picks=Non
         x = x + one_plus_norm(y, t[n + "norm1b"], eps)
         if layer.get("mlp") is not None:
             h = one_plus_norm(x, t[n + "norm2"], eps)
-            y = experts(h, t, layer["mlp"], n + "mlp.", picks=None if picks is None else picks.get(i))
+            y, chosen = experts(h, t, layer["mlp"], n + "mlp.", picks=None if picks is None else picks.get(i))
+            if picks_out is not None:
+                picks_out[i] = chosen
             y = y * sigmoid(h @ t[n + "rg2"].T + t[n + "rg2.b"])
             x = x + one_plus_norm(y, t[n + "norm2b"], eps)
         history.append(x)
