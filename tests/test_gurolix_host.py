@@ -171,3 +171,35 @@ def test_a_pending_update_does_not_pretend_to_be_a_delta():
     assert torch.allclose(delta.total(torch.zeros(2, 4)), torch.ones(2, 4), atol=1e-5)
     with pytest.raises(KernelError):
         delta.dense()
+
+
+def test_bench_design_option_builds_both_models_at_equal_size():
+    import bench
+    name, ours_of, (other, theirs_of), _ = bench.DESIGNS["gurolix"]
+    assert name == "Gurolix" and other == "lfm2_moe_alternating"
+    for width, layers, ff in bench.DESIGN_SIZES.values():
+        ours, theirs = build_model(ours_of(width, layers, ff), "bfloat16"), build_model(theirs_of(width, layers, ff), "bfloat16")
+        assert len(ours.run) == len(theirs.run) == layers and ours.spec.hidden_size == theirs.spec.hidden_size == width
+        for mine, theirs_block in zip(ours.blocks, theirs.blocks):
+            attends = type(mine.mixer).__name__ == "RotaryAttention"
+            assert attends == (type(theirs_block.mixer).__name__ == "Attention")
+            if attends:
+                assert (mine.mixer.num_heads, mine.mixer.num_kv_heads, mine.mixer.head_dim) == \
+                       (theirs_block.mixer.num_heads, theirs_block.mixer.num_kv_heads, theirs_block.mixer.head_dim)
+        routed, theirs_routed = ours.blocks[1].ffn, theirs.blocks[1].ffn
+        assert routed.num_experts + routed.identity == theirs_routed.num_experts and routed.top_k == theirs_routed.top_k
+        assert routed.intermediate_size == theirs_routed.intermediate_size
+
+
+def test_an_output_gate_rides_in_its_mixers_projection():
+    tensors = cases.draw_weights(cases.MIXED, 4)
+    model = build_model(cases.MIXED, "bfloat16")
+    load_tensors(model, tensors, "cpu")
+    for i, block in enumerate(model.blocks):
+        gate, col = block.gates[0], block.gates[0]._rides[1]
+        assert gate.weight is None and col % 16 == 0
+        assert torch.equal(block.mixer.w_in[col:col + 44], tensors[f"l{i}.rg1"])
+        if getattr(block.mixer, "proj_bias", None) is not None:
+            assert block.mixer.proj_bias.shape[0] == block.mixer.w_in.shape[0] and not block.mixer.proj_bias[col:].any()
+        if block.ffn is not None:
+            assert torch.equal(block.gates[1].weight, tensors[f"l{i}.rg2"])
