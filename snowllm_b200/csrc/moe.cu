@@ -32,6 +32,10 @@
 // Bits 8..17 and 20..29: the experts form that many equal groups of neighbours (0 or 1: no groups), and only experts
 // of the best so many groups can be picked; a group's score is the largest score in it (ties to the lower group).
 #define ROUTE_CORRECTED 8
+// Bit 4: a group's score is the sum of its two largest scores instead.  Bit 5: what joins the sum that renormalises the
+// picks' weights is 1e-20 instead of 1e-6.
+#define ROUTE_GROUP_TOP2 16
+#define ROUTE_RENORM_TINY 32
 #define ROUTE_MAX_GROUPS 128
 __host__ __device__ __forceinline__ int route_groups(int flags) { return (flags >> 8) & 0x3ff; }
 __host__ __device__ __forceinline__ int route_groups_kept(int flags) { return (flags >> 20) & 0x3ff; }
@@ -90,9 +94,23 @@ __device__ __forceinline__ void select_topk(float* prob, float* score, int* ids,
 #pragma unroll
     for (int i = 0; i < GR; ++i) best[i] = -INFINITY;
     for (int g = 0; g < count; ++g) {
-      float mx = -INFINITY;
-      for (int e = lane; e < size; e += 32) mx = fmaxf(mx, score[g * size + e]);
-      mx = warp_max(mx);
+      float mx = -INFINITY, second = -INFINITY;
+      for (int e = lane; e < size; e += 32) {
+        const float s = score[g * size + e];
+        second = fmaxf(second, fminf(mx, s));
+        mx = fmaxf(mx, s);
+      }
+      if (flags & ROUTE_GROUP_TOP2) {
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {               // the two largest of two disjoint sets of scores
+          const float om = __shfl_xor_sync(0xffffffffu, mx, o), os = __shfl_xor_sync(0xffffffffu, second, o);
+          second = fmaxf(fmaxf(second, os), fminf(mx, om));
+          mx = fmaxf(mx, om);
+        }
+        if (size > 1) mx += second;
+      } else {
+        mx = warp_max(mx);
+      }
 #pragma unroll
       for (int i = 0; i < GR; ++i)
         if (g == lane + 32 * i) best[i] = mx;
@@ -158,7 +176,7 @@ __device__ __forceinline__ void select_topk(float* prob, float* score, int* ids,
       }
     }
   }
-  const float mul = picked ? 1.f / wsum : (norm_topk ? 1.f / (wsum + 1e-6f) : 1.f);
+  const float mul = picked ? 1.f / wsum : (norm_topk ? 1.f / (wsum + (flags & ROUTE_RENORM_TINY ? 1e-20f : 1e-6f)) : 1.f);
   if (k <= 32) {                   // one round: every pick is in a lane's registers; written once, normalised
     if (lane < k) {
       ids[lane] = my_id;

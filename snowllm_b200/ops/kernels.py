@@ -115,7 +115,15 @@ _SIGNATURES = {
         "snk_mlstm": [P, LL, I, I, I, I, I, P, P, I, F, P, P, P, P, P, P, P, I, I, I, I, P],
     },
     "decay_memory": {
-        "snk_decay_memory": [P, LL, I, I, I, I, P, P, I, P, P, I, F, P, P, P, P, P, P, I, I, I, I, P, P, I, P, P, P, I, P],
+        "snk_decay_memory": [P, LL, I, I, I, I, P, P, I, P, P, I, F, P, P, P, P, P, P, I, I, I, I, P, P, I, P, P, P, I, P, LL, F,
+                             F, P],
+    },
+    "layer_norm": {
+        "snk_layer_norm": [P, P, P, F, F, P, P, P, I, P, F, P, F, F, P, P, I, I, I, P],
+        "snk_side_gate": [P, P, LL, I, P, P, I, P, I, I, I, I, P],
+    },
+    "delta_memory": {
+        "snk_delta_memory": [P, LL, I, I, I, P, LL, P, P, P, LL, F, F, P, P, P, P, P, I, I, I, I, I, I, I, P],
     },
     "streams": {
         "snk_streams_norm": [P, P, P, P, P, P, P, I, P, P, P, P, I, I, F, P, P, I, I, I, I, I, P],
@@ -336,13 +344,26 @@ class DeltaSum:
     A norm that knows it adds both into the residual itself; ``dense()`` forms the sum for anyone else."""
 
     def __init__(self, a, b, a_gate=None):
-        self.a, self.b, self.a_gate = a, b, a_gate
+        self.a = a.dense() if isinstance(a, WeightedSum) else a
+        self.b, self.a_gate = b, a_gate
         self.shape = tuple(a.shape)
 
     def dense(self) -> torch.Tensor:
         out = self.a.clone() if self.a_gate is None else self.a * torch.sigmoid(self.a_gate[:, :1])
         residual_add(out, self.b.dense() if isinstance(self.b, ExpertSum) else self.b)
         return out
+
+
+class WeightedSum:
+    """A residual delta that is ``ca * a + cb * b`` of two float tensors [M, H] (two mixers side by side).  The layer norm
+    forms it in its own kernel; ``dense()`` forms it for anyone else."""
+
+    def __init__(self, a, b, ca: float, cb: float):
+        self.a, self.b, self.ca, self.cb = a, b, float(ca), float(cb)
+        self.shape = tuple(a.shape)
+
+    def dense(self) -> torch.Tensor:
+        return torch.add(self.a * self.ca, self.b, alpha=self.cb)
 
 
 def _pieces_with_rows(delta) -> bool:
@@ -377,8 +398,12 @@ def add_rmsnorm(residual: torch.Tensor, delta, gamma: torch.Tensor, eps: float,
     dscale = 1.0
     if isinstance(delta, NormedDelta):
         return sandwich_norm(residual, delta, gamma, eps, dtype, rows=rows, out=out)
+    if isinstance(delta, WeightedSum):
+        delta = delta.dense()
     if isinstance(delta, ScaledDelta):
         delta, dscale = delta.delta, delta.scale
+        if isinstance(delta, WeightedSum):
+            delta = delta.dense()
     if isinstance(delta, DeltaSum):
         if H % 4 == 0 and _pieces_with_rows(delta.b) and isinstance(delta.a, torch.Tensor):
             moe, gate, delta = delta.b, delta.a_gate, delta.a
@@ -1124,26 +1149,36 @@ ROUTE_GEMM_MIN_ROWS = 64
 ROUTER_SCORINGS = ("sigmoid", "softmax", "softmax_picked")
 
 
-def _route_flags(norm_topk_prob, scoring: str, bias=None, groups=(1, 1)) -> int:
+GROUP_SCORES = ("max", "top2")
+RENORM_EPS = (1e-6, 1e-20)
+
+
+def _route_flags(norm_topk_prob, scoring: str, bias=None, groups=(1, 1), group_score: str = "max",
+                 renorm_eps: float = 1e-6) -> int:
     """The routing kernels' ``norm_topk`` argument: bit 0 renormalises the picks' weights by their sum, bit 1
     scores with a softmax over all experts instead of a sigmoid per expert, bit 2 ("softmax_picked") picks by
     the logits themselves (the bias then belongs to the logit) and weights by the softmax over the picked
     logits alone, bit 3 (a softmax with a ``bias``) adds the bias to the scores that choose.  ``groups`` = (count,
-    keep): only experts of the best ``keep`` of ``count`` equal groups of neighbours can be picked."""
+    keep): only experts of the best ``keep`` of ``count`` equal groups of neighbours can be picked, by a group's largest
+    score or (``group_score`` "top2") by the sum of its two largest.  ``renorm_eps`` joins the renormalising sum."""
+    if group_score not in GROUP_SCORES or renorm_eps not in RENORM_EPS:
+        raise KernelError(f"group score {group_score!r}, renormalisation {renorm_eps}")
     if scoring not in ROUTER_SCORINGS:
         raise KernelError(f"router scoring {scoring!r} (known: {', '.join(ROUTER_SCORINGS)})")
     count, keep = groups
     limits = (int(count) << 8 | int(keep) << 20) if count > 1 else 0
+    limits |= (16 if group_score == "top2" else 0) | (32 if renorm_eps == 1e-20 else 0)
     if scoring == "softmax_picked":
         return 4 | limits
     softmax = (2 | (8 if bias is not None else 0)) if scoring == "softmax" else 0
     return int(bool(norm_topk_prob)) | softmax | limits
 
 
-def moe_route(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring: str = "sigmoid", groups=(1, 1)):
+def moe_route(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring: str = "sigmoid", groups=(1, 1), **choice):
     """(ids int32 [M, k], weights float [M, k]) of the router, computed in float: a sigmoid per expert, or
     (``scoring`` "softmax") a softmax over all experts' logits; the k largest of score + ``bias`` are picked, among
-    the experts of the best ``groups[1]`` of ``groups[0]`` equal groups; the weights are the scores."""
+    the experts of the best ``groups[1]`` of ``groups[0]`` equal groups; the weights are the scores.
+    ``choice``: ``group_score`` and ``renorm_eps`` of ``_route_flags``."""
     M, H = x.shape
     dtype = x.dtype
     _chk(x, "router input", (torch.float32, torch.bfloat16))
@@ -1152,7 +1187,7 @@ def moe_route(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring: str = 
     _chk(router_w, "router weight", shape=(E, H))
     if bias is not None:
         _chk(bias, "expert bias", torch.float32, (E,))
-    flags = _route_flags(norm_topk_prob, scoring, bias, groups)
+    flags = _route_flags(norm_topk_prob, scoring, bias, groups, **choice)
     ids = torch.empty(M, top_k, dtype=torch.int32, device=x.device)
     wts = torch.empty(M, top_k, dtype=torch.float32, device=x.device)
     if (M > ROUTE_GEMM_MIN_ROWS and router_w.dtype == torch.bfloat16 and gemm_tc_ok(x, router_w)
@@ -1186,14 +1221,14 @@ ROUTE_FUSED_MAX_ROWS = 32      # up to here: logits spread over the GPU, selecti
 
 
 def moe_route_sort(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring: str = "sigmoid", groups=(1, 1),
-                   identity: int = 0):
+                   identity: int = 0, **choice):
     """Routing and the sort by expert together: (ids, weights, offsets, pair_pos, sorted_pair) as
     `moe_route` and `moe_sort` give them.  The few rows of a decode step take two launches made for
     them; a row's logits are the same numbers on every path but the tensor-core one."""
     M, H = x.shape
     E = router_w.shape[0]
     if M > ROUTE_FUSED_MAX_ROWS or 8 * E * min(M, 32) + 8 * M * top_k > 48 * 1024:
-        ids, wts = moe_route(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring, groups)
+        ids, wts = moe_route(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring, groups, **choice)
         return (ids, wts) + moe_sort(ids, E, identity)
     dtype = x.dtype
     _chk(x, "router input", (torch.float32, torch.bfloat16))
@@ -1210,7 +1245,7 @@ def moe_route_sort(x, router_w, bias, top_k, norm_topk_prob, scaling, scoring: s
     logits, wts = floats[:M * E], floats[M * E:].view(M, top_k)
     check(fn("snk_moe_route_sort")(_ptr(x), _ptr(router_w), w32, _ptr(bias), _ptr(logits), _ptr(ids), _ptr(wts),
                                    _ptr(offsets), _ptr(pair_pos), _ptr(sorted_pair), M, H, E, E - int(identity), top_k,
-                                   _route_flags(norm_topk_prob, scoring, bias, groups), float(scaling), code_of(dtype),
+                                   _route_flags(norm_topk_prob, scoring, bias, groups, **choice), float(scaling), code_of(dtype),
                                    _stream()),
           "moe_route_sort", launches=2, work=lambda: (_nbytes(x, router_w, ints, floats), 2 * M * E * H))
     return ids, wts, offsets, pair_pos, sorted_pair
@@ -1491,7 +1526,7 @@ def add_dyt(residual, delta, weight, bias, alpha, dtype, rows=None, out=None):
     M, H = residual.shape
     _chk(residual, "residual", torch.float32)
     da = db = moe = None
-    if isinstance(delta, ScaledDelta) or (isinstance(delta, DeltaSum) and delta.a_gate is not None):
+    if isinstance(delta, (ScaledDelta, WeightedSum)) or (isinstance(delta, DeltaSum) and delta.a_gate is not None):
         delta = delta.dense()              # a factor or a gate per row: forms this kernel does not apply itself
     if isinstance(delta, DeltaSum):
         da, db = delta.a, delta.b
@@ -1718,7 +1753,7 @@ def sandwich_norm(residual, delta: NormedDelta, weight, eps, dtype, *, rows=None
     _chk(residual, "residual", torch.float32)
     _chk(weight, "norm weight", torch.float32, (W,))
     y, moe = delta.y, None
-    if isinstance(y, (ScaledDelta, DeltaSum)):
+    if isinstance(y, (ScaledDelta, DeltaSum, WeightedSum)):
         y = y.dense()
     if isinstance(y, ExpertSum):
         moe, y = y, y.y
@@ -1764,6 +1799,85 @@ def sandwich_norm(residual, delta: NormedDelta, weight, eps, dtype, *, rows=None
                                    + (delta.history is not None and rows is None)
                                    + (delta.index if delta.average is not None else 0))
                       + (R * W * out.element_size() if delta.gate is not None else 0) + _nbytes(out), 0))
+    return out
+
+
+# --- layer norm; side inputs from the token ids ------------------------------------------------------
+
+def layer_norm(residual, delta, weight, eps, dtype, *, gain: float = 1.0, rows=None, out=None):
+    """``residual += delta``, then the layer norm of the sum (centred, ``weight`` float [H], times ``gain``) in
+    ``dtype``; ``weight`` None: the sum itself in ``dtype``.  ``delta``: None, a float tensor, an ``ExpertSum``, a
+    ``WeightedSum``, a ``DeltaSum`` or ``ScaledDelta`` of these, or a ``NormedDelta`` with a norm of its own (no gate, no
+    history).  With ``rows`` only those rows come out and the residual stays as it is."""
+    M, W = residual.shape
+    _chk(residual, "residual", torch.float32)
+    w1, eps1 = None, 0.0
+    if isinstance(delta, NormedDelta):
+        if delta.gate is not None or delta.history is not None or delta.weight is None or delta.y is None:
+            raise KernelError("the layer norm applies a pending update with a norm of its own, not with a gate or a "
+                              "history")
+        w1, eps1, delta = delta.weight, delta.eps, delta.y
+        _chk(w1, "update's norm weight", torch.float32, (W,))
+    a = b = moe = None
+    ca = cb = 1.0
+    if isinstance(delta, WeightedSum):
+        a, b, ca, cb = delta.a, delta.b, delta.ca, delta.cb
+    elif isinstance(delta, DeltaSum) and delta.a_gate is None and torch.is_tensor(delta.a):
+        a = delta.a
+        if _pieces_with_rows(delta.b):
+            moe = delta.b
+        else:
+            b = delta.b.dense() if hasattr(delta.b, "dense") else delta.b
+    elif _pieces_with_rows(delta):
+        moe = delta
+    elif isinstance(delta, ScaledDelta):
+        a, ca = (delta.delta.dense() if hasattr(delta.delta, "dense") else delta.delta), delta.scale
+    elif delta is not None:
+        a = delta.dense() if hasattr(delta, "dense") else delta
+    for name, t in (("residual delta", a), ("second residual delta", b)):
+        if t is not None:
+            _chk(t, name, torch.float32, (M, W))
+    k = 0
+    if moe is not None:
+        k = moe.weights.shape[1]
+        _chk(moe.y, "expert outputs", torch.float32)
+        _chk(moe.pair_pos, "pair positions", torch.int32, (M * k,))
+        _chk(moe.weights, "top-k weights", torch.float32)
+    if weight is not None:
+        _chk(weight, "norm weight", torch.float32, (W,))
+    R = M if rows is None else rows.numel()
+    if rows is not None:
+        _chk(rows, "norm rows", torch.int32)
+    if out is None:
+        out = torch.empty(R, W, dtype=dtype, device=residual.device)
+    _chk(out, "norm output", dtype, (R, W))
+    terms = (a is not None) + (b is not None) + k
+    check(fn("snk_layer_norm")(
+        _ptr(residual), _ptr(a), _ptr(b), float(ca), float(cb), _ptr(moe.y if moe else None),
+        _ptr(moe.pair_pos if moe else None), _ptr(moe.weights if moe else None), k, _ptr(w1), float(eps1), _ptr(weight),
+        float(eps), float(gain), _ptr(out), _ptr(rows), R, W, code_of(dtype), _stream()), "layer_norm",
+        work=lambda: (R * W * 4 * (1 + terms + (terms > 0 and rows is None)) + _nbytes(out), 0))
+    return out
+
+
+def side_gate(g, table, ids, col: int, dtype, pending=None, out=None):
+    """gelu(g) * table[id, col : col + n] in ``dtype``: ``g`` float [M, n] (gelu in its tanh form), ``table`` [vocab,
+    width] in ``dtype``, ``ids`` int32 [M] (an id -(i + 1) reads its token from ``pending[i]``)."""
+    M, n = g.shape
+    _chk(g, "side gate", torch.float32)
+    _chk(table, "side table", dtype)
+    _chk(ids, "side ids", torch.int32, (M,))
+    if col < 0 or col + n > table.shape[1]:
+        raise KernelError(f"a side table of width {table.shape[1]} holds no {n} columns from {col} on")
+    if pending is not None:
+        _chk(pending, "pending tokens", torch.int32)
+    if out is None:
+        out = torch.empty(M, n, dtype=dtype, device=g.device)
+    _chk(out, "side output", dtype, (M, n))
+    check(fn("snk_side_gate")(_ptr(g), _ptr(table), table.shape[1], int(col), _ptr(ids), _ptr(pending),
+                              pending.numel() if pending is not None else 0, _ptr(out), M, n, table.shape[0],
+                              code_of(dtype), _stream()), "side_gate",
+          work=lambda: (_nbytes(g, out, ids) + M * n * table.element_size(), 0))
     return out
 
 
@@ -2054,13 +2168,15 @@ def mlstm(proj, q_off, k_off, v_off, i_off, f_off, bias_i, bias_f, cap, cu_seqle
 
 def decay_memory(proj, q_off, k_off, v_off, cu_seqlens, seg_start, seg_slot, state, heads, dk, dv, *,
                  gate_bias=None, gate_low=None, decay=None, inv_freq=None, rot_dim=0, k_scale=1.0, positions=None,
-                 out=None, pieces=None):
+                 out=None, pieces=None, z=None, z_col=0, sharp=1.0, q_scale=1.0):
     """S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per (segment, head) over a flat batch.  ``proj``:
     float [M, width] with q at ``q_off`` and k (or the gate's pre-activation) at ``k_off`` ([heads, dk] each)
     and v at ``v_off`` ([heads, dv]).  Gated form (``gate_bias`` and ``gate_low`` over [heads*dk]): f = low +
     (1 - low) * sigmoid(z + bias), a = f, k = 1 - f, q = silu(projection).  Fixed form (``decay`` float
     [heads]): a = decay[head] for every row; the first ``rot_dim`` elements of q and k of each head turn with
-    ``positions`` (split halves, ``inv_freq`` float [rot_dim/2]); k times ``k_scale`` afterwards.  ``state``
+    ``positions`` (split halves, ``inv_freq`` float [rot_dim/2]); k times ``k_scale`` afterwards.  Channel form (``z``
+    float [M, width'], heads*dk columns from ``z_col`` on, and ``gate_bias``): a = sigmoid(z + bias)^sharp, q times
+    ``q_scale``.  ``state``
     (float [slots, heads, dk, dv]) is read unless a segment starts at 0, and brought up to date.  Returns
     the raw head outputs, float [M, heads*dv].  ``pieces`` = (int32 [n, 4] = segment, first row, rows, flags
     with 1 for a segment's first piece and 2 for its last; int32 [B+1] = first piece of each segment): every
@@ -2074,9 +2190,19 @@ def decay_memory(proj, q_off, k_off, v_off, cu_seqlens, seg_start, seg_slot, sta
     _chk(state, "memory state", torch.float32, (state.shape[0], heads, dk, dv))
     if width < max(q_off + heads * dk, k_off + heads * dk, v_off + heads * dv):
         raise KernelError(f"memory projection of width {width} is too narrow")
-    gated = gate_bias is not None
+    channel = z is not None
+    gated = gate_bias is not None and not channel
     g32 = 0
-    if gated:
+    z_ptr, z_ld = c_void_p(0), 0
+    if channel:
+        g32 = _small(gate_bias, "decay bias", torch.float32)
+        _chk(gate_bias, "decay bias", shape=(heads * dk,))
+        _chk(z, "decay rows", torch.float32)
+        if z.dim() != 2 or z.shape[0] != M or z.shape[1] < z_col + heads * dk:
+            raise KernelError(f"decay rows of shape {tuple(z.shape)} hold no {heads * dk} columns from {z_col} on")
+        z_ptr, z_ld = c_void_p(z.data_ptr() + 4 * z_col), z.shape[1]
+        inv_freq, rot_dim = None, 0
+    elif gated:
         g32 = _small(gate_bias, "gate bias", torch.float32)
         if gate_low is None or _small(gate_low, "gate lower bound", torch.float32) != g32:
             raise KernelError("gate bias and lower bound must both be given, in one dtype")
@@ -2103,13 +2229,14 @@ def decay_memory(proj, q_off, k_off, v_off, cu_seqlens, seg_start, seg_slot, sta
         _chk(cu_pieces, "first piece of each segment", torch.int32, (B + 1,))
         work = torch.empty(n_pieces, heads, dk, dv, dtype=torch.float32, device=proj.device)
         work_decay = torch.empty(n_pieces, heads, dk, dtype=torch.float32, device=proj.device)
-        prep = torch.empty(3 if gated else 2, M, heads * dk, dtype=torch.float32, device=proj.device)
-    check(fn("snk_decay_memory")(_ptr(proj), width, q_off, k_off, v_off, 0 if gated else 1, _ptr(gate_bias),
+        prep = torch.empty(3 if gated or channel else 2, M, heads * dk, dtype=torch.float32, device=proj.device)
+    check(fn("snk_decay_memory")(_ptr(proj), width, q_off, k_off, v_off, 2 if channel else (0 if gated else 1), _ptr(gate_bias),
                                  _ptr(gate_low), g32, _ptr(decay), _ptr(inv_freq), int(rot_dim), float(k_scale),
                                  _ptr(positions), _ptr(cu_seqlens), _ptr(seg_start), _ptr(seg_slot), _ptr(state),
                                  _ptr(out), B, heads, dk, dv, _ptr(table), _ptr(cu_pieces), n_pieces, _ptr(work),
-                                 _ptr(work_decay), _ptr(prep), M, _stream()), "decay_memory",
-          launches=4 if n_pieces else 1, work=lambda: _decay_memory_work(M, B, heads, dk, dv, n_pieces, gated))
+                                 _ptr(work_decay), _ptr(prep), M, z_ptr, z_ld, float(sharp),
+                                 float(q_scale), _stream()), "decay_memory",
+          launches=4 if n_pieces else 1, work=lambda: _decay_memory_work(M, B, heads, dk, dv, n_pieces, gated or channel))
     return out
 
 
@@ -2124,6 +2251,46 @@ def _decay_memory_work(M, B, H, dk, dv, pieces, gated):
             (prep - rows_k + rows_v + pieces * cells * 4, 3 * M * cells),
             (2 * pieces * cells * 4 + B * cells * 4, 2 * pieces * cells),
             (prep + 2 * rows_v + pieces * cells * 4 + B * cells * 4, 5 * M * cells)]
+
+
+def delta_memory(u, q_off, k_off, v_off, z, z_col, bias, rate, beta, beta_col, cu_seqlens, seg_start, seg_slot, state,
+                 kv_heads, max_len, *, unit_eps: float, q_scale: float, out=None):
+    """The gated delta rule: S <- diag(a_t) S; w = sigmoid(beta_t) (v_t - S^T k_t); S <- S + k_t w^T; o_t = S^T q_t per
+    (segment, head) over a flat batch.  ``u`` [M, width] (compute dtype) holds q and k [kv_heads, dk] at ``q_off`` and
+    ``k_off``, made unit vectors here (``unit_eps`` joins the squared length; q times ``q_scale``), and v [heads, dv] at
+    ``v_off``; a = exp(rate[h] softplus(z + bias)) with ``z`` float [M, width'], heads*dk columns from ``z_col`` on,
+    ``bias`` float [heads*dk] and ``rate`` (negative) float [heads]; ``beta`` [M, width''] (compute dtype): a logit per
+    head from ``beta_col`` on.  ``state`` float [slots, heads, dk, dv] is read unless a segment starts at 0, and brought
+    up to date.  ``max_len``: the longest segment.  Returns float [M, heads * dv]."""
+    M, width = u.shape
+    dtype = u.dtype
+    _chk(u, "memory rows", (torch.float32, torch.bfloat16))
+    slots, H, dk, dv = state.shape
+    _chk(state, "memory state", torch.float32)
+    if width < max(q_off + kv_heads * dk, k_off + kv_heads * dk, v_off + H * dv):
+        raise KernelError(f"memory rows of width {width} are too narrow")
+    _chk(z, "decay rows", torch.float32)
+    _chk(beta, "write strengths", dtype)
+    for name, t, need in (("decay rows", z, z_col + H * dk), ("write strengths", beta, beta_col + H)):
+        if t.dim() != 2 or t.shape[0] != M or t.shape[1] < need:
+            raise KernelError(f"{name} of shape {tuple(t.shape)}, want [{M}, at least {need}]")
+    _chk(bias, "decay bias", torch.float32, (H * dk,))
+    _chk(rate, "decay rate", torch.float32, (H,))
+    B = seg_start.numel()
+    _chk(cu_seqlens, "cu_seqlens", torch.int32, (B + 1,))
+    _chk(seg_start, "seg_start", torch.int32, (B,))
+    _chk(seg_slot, "seg_slot", torch.int32, (B,))
+    if out is None:
+        out = torch.empty(M, H * dv, dtype=torch.float32, device=u.device)
+    _chk(out, "memory output", torch.float32, (M, H * dv))
+    check(fn("snk_delta_memory")(
+        _ptr(u), width, int(q_off), int(k_off), int(v_off), c_void_p(z.data_ptr() + 4 * z_col), z.shape[1], _ptr(bias),
+        _ptr(rate), c_void_p(beta.data_ptr() + beta_col * beta.element_size()), beta.shape[1], float(q_scale),
+        float(unit_eps), _ptr(cu_seqlens), _ptr(seg_start), _ptr(seg_slot), _ptr(state), _ptr(out), B, H, int(kv_heads),
+        dk, dv, int(max_len), code_of(dtype), _stream()), "delta_memory",
+        work=lambda: ((2 * kv_heads * dk + H * dv) * M * u.element_size() + M * H * (dk * 4 + u.element_size())
+                      + _nbytes(out) + 2 * B * H * dk * dv * 4, 7 * M * H * dk * dv))
+    return out
 
 
 # --- several residual streams ------------------------------------------------------------------------
@@ -2165,7 +2332,7 @@ def streams_norm(streams, weight, groups, eps, dtype, *, init=None, update: Stre
         if update.streams is not streams:
             raise KernelError("the pending update belongs to other streams")
         y = update.y
-        if isinstance(y, ScaledDelta) or (isinstance(y, DeltaSum) and y.a_gate is not None):
+        if isinstance(y, (ScaledDelta, WeightedSum)) or (isinstance(y, DeltaSum) and y.a_gate is not None):
             y = y.dense()                  # a factor or a gate per row: forms this kernel does not apply itself
         if isinstance(y, DeltaSum):
             da, y = y.a, y.b

@@ -28,8 +28,9 @@ Six kinds are built on one class:
   score is 0 and which has no value); each head's output times sigmoid of the head's own logit from a gate
   projection [heads, hidden] that reads the mixer's input.
 
-* ``rotary_attention``: causal, biased projections, optional per-head norms, rotary positions, optionally a cap on
-  the scores and values mixed with those of the first layer that mixes (``RotaryAttention``).
+* ``rotary_attention``: causal, projections with or without biases, optional per-head norms, rotary positions in either
+  layout, optionally a sink per head, the projected keys as values, a cap on the scores and values mixed with those of
+  the first layer that mixes (``RotaryAttention``).
 
 The first two: per-head RMS norm of q and k with one weight of ``head_dim`` shared by all heads (and maps), before
 the rotation; ``window`` keeps the last ``window`` keys.  Scores, softmax weights and the per-head
@@ -48,6 +49,7 @@ from ..errors import ConfigError, KernelError
 from ..ops import kernels, linear
 from . import attention_plan as plan
 from .base import Part
+from .position import halves_order
 from .registry import lookup, register_mixer
 from .spec import INIT_BIAS, INIT_CONV, INIT_ONES, KEEP_F32, KEEP_SMALL, PagedKVSpec, SlotStateSpec, TensorSpec
 
@@ -124,6 +126,7 @@ class MapsAttention(Part):
     whole_norm = False         # True: ONE root mean square over all heads of q (of k), weights of that size
     keep_first = 0             # positions at the sequence's start that stay reachable beside the window
     _lends_rows = False        # whether the fused projection carries rows of another part (``append_input_rows``)
+    keys_are_values = False    # the values are the projected keys, as they are before norm and rotation
     softcap = None             # c: a scaled score s becomes c * tanh(s / c)
 
     def __init__(self, dtype, names, *, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int,
@@ -167,6 +170,9 @@ class MapsAttention(Part):
         """(q, k, v, gate) column offsets of the fused projection, and its width."""
         q = 0
         k = q + self.nq * self.head_dim
+        if self.keys_are_values:
+            g = k + self.num_kv_heads * self.head_dim
+            return q, k, k, g, g + self._gate_width()
         v = k + (0 if self.reads_cache else self.num_kv_heads * self.maps * self.head_dim)
         g = v + (0 if self.reads_cache else self.num_kv_heads * self.v_head_dim)
         return q, k, v, g, g + self._gate_width()
@@ -182,8 +188,9 @@ class MapsAttention(Part):
         H, dk, dv, n = self.hidden_size, self.head_dim, self.v_head_dim, self.names
         specs = [TensorSpec("q_proj", n["q_proj"], (self.nq * dk, H))]
         if not self.reads_cache:
-            specs += [TensorSpec("k_proj", n["k_proj"], (self.num_kv_heads * self.maps * dk, H)),
-                      TensorSpec("v_proj", n["v_proj"], (self.num_kv_heads * dv, H))]
+            specs.append(TensorSpec("k_proj", n["k_proj"], (self.num_kv_heads * self.maps * dk, H)))
+            if not self.keys_are_values:
+                specs.append(TensorSpec("v_proj", n["v_proj"], (self.num_kv_heads * dv, H)))
         specs.append(TensorSpec("out_proj", n["out_proj"], (H, self.num_heads * dv)))
         if self.qk_norm_eps is not None and self.norm_weights:
             nq, nk = (self.nq * dk, self.num_kv_heads * self.maps * dk) if self.whole_norm else (dk, dk)
@@ -195,7 +202,7 @@ class MapsAttention(Part):
     def _projection_rows(self, tensors) -> list:
         rows = [tensors["q_proj"]]
         if not self.reads_cache:
-            rows += [tensors["k_proj"], tensors["v_proj"]]
+            rows += [tensors["k_proj"]] + ([] if self.keys_are_values else [tensors["v_proj"]])
         return rows
 
     def bind(self, tensors):
@@ -532,15 +539,19 @@ class ConvGateAttention(MapsAttention):
 
 
 class RotaryAttention(MapsAttention):
-    """One map per head; projections with biases; per-head RMS norm of q and k (``qk_norm_eps`` None: none) before the
-    rotation; ``softcap`` c on the scaled scores; and values that go over into those of an earlier layer: with
+    """One map per head; projections with biases (``biased`` False: without); per-head RMS norm of q and k (``qk_norm_eps``
+    None: none; ``qk_norm_weights`` False: the plain root mean square) before the rotation, which for the plain root mean
+    square is the same as after it: a rotation keeps a head's length; rotary positions in halves or in pairs (then the
+    rows of the projections are laid out in halves when they are bound); ``with_sink``: one more term exp(sink) per head in
+    the softmax's sum; ``keys_are_values``: the values are the projected keys, before norm and rotation, and there is no
+    value projection; ``softcap`` c on the scaled scores; and values that go over into those of an earlier layer: with
     ``value_mix`` "first" the layer leaves its values in the step's memo, with "mix" it caches (1 - lambda) v +
     lambda v_first (lambda a learned number, ``value_mix`` among its tensors in either role)."""
     libraries = MapsAttention.libraries + ("attention_tc", "attention_mma")
     VALUES = "first_values"            # the memo key under which the first mixing layer's values are found
 
     def __init__(self, dtype, names, *, softcap: float | None = None, value_mix: str | None = None, biased: bool = True,
-                 **kw):
+                 qk_norm_weights: bool = True, with_sink: bool = False, keys_are_values: bool = False, **kw):
         super().__init__(dtype, names, **kw)
         if softcap is not None and not softcap > 0:
             raise ConfigError(f"a score cap of {softcap}: want a positive number")
@@ -548,6 +559,9 @@ class RotaryAttention(MapsAttention):
             raise ConfigError(f"value_mix={value_mix!r} (known: first, mix)")
         if self.reads_cache and value_mix is not None:
             raise ConfigError("a layer that reads another layer's cache has no values to mix")
+        if keys_are_values and (biased or self.reads_cache or value_mix is not None or self.head_dim != self.v_head_dim):
+            raise ConfigError("keys that are the values have their width, no biases, and a cache and values of their own")
+        self.norm_weights, self.with_sink, self.keys_are_values = bool(qk_norm_weights), bool(with_sink), bool(keys_are_values)
         self.softcap, self.value_role, self.biased = softcap, value_mix, biased
         self.value_lambda = 0.0
 
@@ -560,10 +574,33 @@ class RotaryAttention(MapsAttention):
                       TensorSpec("v_bias", n["v_bias"], (self.num_kv_heads * dv,), INIT_BIAS, KEEP_F32)]
         if self.value_role is not None:
             specs.append(TensorSpec("value_mix", n["value_mix"], (), INIT_BIAS, KEEP_F32))
+        if self.with_sink:
+            specs.append(TensorSpec("sink", n["sink"], (self.num_heads,), INIT_BIAS, KEEP_F32))
         return specs
 
+    def _in_halves(self, tensors) -> dict:
+        """The tensors with every head's elements in the order in which the pairs that turn together stand half a
+        rotation apart.  Keys that are values take the value heads along, so the output product's columns follow."""
+        order = torch.tensor(halves_order(self.head_dim, self.position.rot_dim))
+        d, out = self.head_dim, dict(tensors)
+
+        def reorder(t, heads):                     # rows [heads * d, ...]
+            at = (torch.arange(heads)[:, None] * d + order[None, :]).reshape(-1).to(t.device)
+            return t.index_select(0, at).contiguous()
+        for name, heads in (("q_proj", self.num_heads), ("k_proj", self.num_kv_heads), ("q_bias", self.num_heads),
+                            ("k_bias", self.num_kv_heads), ("q_norm", 1), ("k_norm", 1)):
+            if name in out:
+                out[name] = reorder(out[name], heads)
+        if self.keys_are_values:
+            out["out_proj"] = reorder(out["out_proj"].t(), self.num_heads).t().contiguous()
+        return out
+
     def bind(self, tensors):
+        if getattr(self.position, "layout", "halves") == "pairs":
+            tensors = self._in_halves(tensors)
         super().bind(tensors)
+        if self.with_sink:
+            self.sink = tensors["sink"].float().contiguous()
         if self.biased:
             bias = torch.cat([tensors[k].float() for k in ("q_bias", "k_bias", "v_bias")])
             self.proj_bias = torch.cat((bias, bias.new_zeros(self.w_in.shape[0] - bias.numel()))).contiguous()

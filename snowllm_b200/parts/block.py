@@ -27,22 +27,38 @@ from .base import Part
 from ..ops import linear
 from .registry import lookup, register_block
 from .spec import INIT_BIAS, KEEP_F32, TensorSpec
+from .token_side import TokenSide
 
 
 class PreNormBlock:
     """``residual_scale`` m (a constant of the arrangement): x += m * mixer(norm(x)); x += m * ffn(norm(x)).
-    The factor travels with the delta (``kernels.ScaledDelta``) to the norm that adds it."""
+    The factor travels with the delta (``kernels.ScaledDelta``) to the norm that adds it.
 
-    def __init__(self, mixer, ffn, mixer_norm, ffn_norm, *, dtype=None, residual_scale: float = 1.0):
+    ``side`` (a ``PartSpec`` of parts/token_side.py): after the sublayers the layer adds an input of its own from the
+    token ids; that update is what stays pending for the norm that follows."""
+
+    def __init__(self, mixer, ffn, mixer_norm, ffn_norm, *, dtype=None, residual_scale: float = 1.0, side=None):
         self.mixer, self.ffn, self.mixer_norm, self.ffn_norm = mixer, ffn, mixer_norm, ffn_norm
         self.residual_scale = float(residual_scale)
+        if side is not None and side.kind != "token_side":
+            raise ConfigError(f"a layer's side input of kind {side.kind!r} (known: token_side)")
+        self.side = TokenSide(dtype, side.names, **dict(side.params)) if side is not None else None
         self._names = tuple(f"{what}:{type(part).__name__}" for what, part in
                             (("norm", mixer_norm), ("mixer", mixer), ("norm", ffn_norm), ("ffn", ffn)))
 
     def parts(self):
-        return tuple(p for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn) if p is not None)
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn, self.side) if p is not None)
 
     def forward(self, ctx, residual, delta, cache, owns_cache=True):
+        if self.side is None:
+            return self._sublayers(ctx, residual, delta, cache, owns_cache)
+        delta = self._sublayers(ctx, residual, delta, cache, owns_cache, tap=False)
+        with span("side:TokenSide"):
+            delta = self.side.forward(ctx, residual, delta)
+        self._tap_layer(ctx, residual, delta)
+        return delta
+
+    def _sublayers(self, ctx, residual, delta, cache, owns_cache, tap=True):
         with span(self._names[0]):
             x = self.mixer_norm.forward(ctx, residual, delta)
         ctx.tap("mixer_in", x)
@@ -50,9 +66,10 @@ class PreNormBlock:
             delta = self.mixer.forward(ctx, x, cache, owns_cache)
         ctx.tap("mixer_out", delta)
         if self.residual_scale != 1.0:
-            return self._scaled(ctx, residual, delta)
+            return self._scaled(ctx, residual, delta, tap)
         if self.ffn is None:
-            self._tap_layer(ctx, residual, delta)
+            if tap:
+                self._tap_layer(ctx, residual, delta)
             return delta
         fused = getattr(self.ffn, "forward_from_residual", None)
         if fused is not None:          # a feed-forward that can take the norm before it into its first kernel
@@ -60,7 +77,8 @@ class PreNormBlock:
                 out = fused(ctx, residual, delta, self.ffn_norm)
             if out is not None:
                 ctx.tap("ffn_out", out)
-                self._tap_layer(ctx, residual, out)
+                if tap:
+                    self._tap_layer(ctx, residual, out)
                 return out
         with span(self._names[2]):
             x = self.ffn_norm.forward(ctx, residual, delta)
@@ -68,15 +86,19 @@ class PreNormBlock:
         with span(self._names[3]):
             delta = self.ffn.forward(ctx, x)
         ctx.tap("ffn_out", delta)
-        self._tap_layer(ctx, residual, delta)
+        if tap:
+            self._tap_layer(ctx, residual, delta)
         return delta
 
     @staticmethod
     def _tap_layer(ctx, residual, delta):
         if ctx.taps is not None:
-            ctx.tap("layer_out", residual + (delta.dense() if hasattr(delta, "dense") else delta))
+            if hasattr(delta, "total"):
+                ctx.tap("layer_out", delta.total(residual))
+            else:
+                ctx.tap("layer_out", residual + (delta.dense() if hasattr(delta, "dense") else delta))
 
-    def _scaled(self, ctx, residual, delta):
+    def _scaled(self, ctx, residual, delta, tap=True):
         """The rest of the layer when the sublayers' outputs enter the stream times a constant."""
         delta = kernels.ScaledDelta(delta, self.residual_scale)
         if self.ffn is not None:
@@ -86,7 +108,8 @@ class PreNormBlock:
             with span(self._names[3]):
                 delta = kernels.ScaledDelta(self.ffn.forward(ctx, x), self.residual_scale)
             ctx.tap("ffn_out", delta.delta)
-        self._tap_layer(ctx, residual, delta)
+        if tap:
+            self._tap_layer(ctx, residual, delta)
         return delta
 
 
@@ -114,6 +137,7 @@ class OutputNormBlock:
         ctx.tap("mixer_in", x)
         with span(self._names[0]):
             y = self.mixer.forward(ctx, x, cache, owns_cache)
+        y = y.dense() if hasattr(y, "dense") else y
         ctx.tap("mixer_out", y)
         with span(self._names[1]):
             x = self.mixer_norm.add_normed(ctx, residual, y)

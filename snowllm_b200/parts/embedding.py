@@ -9,34 +9,42 @@ from .base import Part
 from .registry import lookup, register_embedding, register_head
 from ..errors import ConfigError
 from .spec import PartSpec, SlotStateSpec, TensorSpec
+from .token_side import TABLE as SIDE_TABLE
 
 
 class Embedding(Part):
     libraries = ("elementwise",)
 
     def __init__(self, dtype, names, *, vocab_size: int, hidden_size: int, scale: float = 1.0,
-                 norm: PartSpec | None = None):
+                 norm: PartSpec | None = None, side_size: int | None = None):
         """``scale``: a constant that multiplies every row on its way into the stream; ``norm``: a norm the rows pass
-        before they enter it (in float, like the stream)."""
+        before they enter it (in float, like the stream); ``side_size``: the width of a second table of token rows that
+        layers read on their own (parts/token_side.py)."""
         super().__init__(dtype, names)
         self.vocab_size, self.hidden_size, self.scale = vocab_size, hidden_size, float(scale)
-        self.weight = None
+        self.weight = self.side = None
+        self.side_size = side_size
         self.norm = lookup("norm", norm.kind)(torch.float32, norm.names, **dict(norm.params)) if norm else None
 
     def parts(self):
         return (self.norm,) if self.norm is not None else ()
 
     def declare(self, has):
-        return [TensorSpec("weight", self.names["weight"], (self.vocab_size, self.hidden_size))]
+        specs = [TensorSpec("weight", self.names["weight"], (self.vocab_size, self.hidden_size))]
+        if self.side_size:
+            specs.append(TensorSpec("side", self.names["side"], (self.vocab_size, self.side_size)))
+        return specs
 
     def bind(self, tensors):
-        self.weight = tensors["weight"]
+        self.weight, self.side = tensors["weight"], tensors.get("side")
 
     def bytes_read(self, bound, picked=None):
         return 0        # a step gathers one row per token: nothing beside the matrices
 
     def forward(self, ctx):
         """The float residual stream [M, H] of the step's tokens."""
+        if self.side is not None:
+            ctx.memo[SIDE_TABLE] = self.side
         x = kernels.embedding(ctx.token_ids, self.weight, pending=ctx.pending_tokens, scale=self.scale)
         return x if self.norm is None else self.norm.forward(ctx, x)
 

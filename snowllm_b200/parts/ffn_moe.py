@@ -15,7 +15,8 @@ by sigmoid(w_sg . x), one number per token (tensor ``shared_row_gate`` [1, hidde
 "softmax_picked": the router's logits, plus the bias ``expert_bias`` which is then a part of the logit, pick
 the k largest, and the weights are the softmax over the picked logits alone.  With ``scoring`` "softmax" an
 ``expert_bias`` is a correction that only chooses.  ``groups`` (count, keep): the router's outputs form equal groups
-of neighbours, and only experts of the best ``keep`` groups can be chosen.  ``identity``: that many more router
+of neighbours, and only experts of the best ``keep`` groups can be chosen (``group_score`` "max": by a group's largest
+score, "top2": by the sum of its two largest).  ``renorm_eps``: what joins the sum that renormalises the picks' weights.  ``identity``: that many more router
 outputs stand for experts that return their input.  ``gated`` False: an expert is down(act(up x)), ``activation`` one
 of the plain ones (the square of relu among them)."""
 from __future__ import annotations
@@ -36,7 +37,7 @@ class SigmoidMoE(Part):
                  top_k: int, norm_topk_prob: bool, use_expert_bias: bool, routed_scaling_factor: float,
                  scale_input: bool = False, scoring: str = "sigmoid", activation: str = "silu",
                  limit: float | None = None, shared: dict | None = None, gated: bool = True, groups=(1, 1),
-                 identity: int = 0):
+                 identity: int = 0, group_score: str = "max", renorm_eps: float = 1e-6):
         """``scale_input``: a pick's weight multiplies the expert's INPUT (the output is the plain sum of
         expert(w * x) over the picks) instead of its output.  ``shared``: {"intermediate_size", "limit"}."""
         super().__init__(dtype, names)
@@ -59,6 +60,10 @@ class SigmoidMoE(Part):
         if self.groups[0] > 128 or (num_experts + self.identity) % self.groups[0]:
             raise ConfigError(f"{num_experts + self.identity} router outputs in {self.groups[0]} groups (up to 128 equal "
                               f"groups)")
+        if group_score not in kernels.GROUP_SCORES or renorm_eps not in kernels.RENORM_EPS:
+            raise ConfigError(f"group_score={group_score!r}, renorm_eps={renorm_eps} (known: "
+                              f"{', '.join(kernels.GROUP_SCORES)}; {', '.join(map(str, kernels.RENORM_EPS))})")
+        self.choice = dict(group_score=group_score, renorm_eps=renorm_eps)
         self.scoring, self.activation, self.limit = scoring, activation, limit
         self.shared = dict(shared) if shared is not None else None
         self.shared_w13 = self.shared_w2 = self.shared_row_gate = None
@@ -138,7 +143,7 @@ class SigmoidMoE(Part):
 
     def route(self, x):
         return kernels.moe_route(x, self.router, self.bias, self.top_k, self.norm_topk_prob,
-                                 self.routed_scaling_factor, self.scoring, self.groups)
+                                 self.routed_scaling_factor, self.scoring, self.groups, **self.choice)
 
     def forward_from_residual(self, ctx, residual, delta, norm):
         """The norm that precedes this feed-forward, the router and the sort in one launch, for the few rows
@@ -149,7 +154,8 @@ class SigmoidMoE(Part):
             return None
         if self.scale_input or not kernels.FUSE_ROUTER or not kernels.norm_route_sort_ok(residual, delta, weight, self.router, self.top_k):
             return None
-        if self.scoring != "sigmoid" or self.activation != "silu" or self.shared is not None or self.groups[0] > 1:
+        if self.scoring != "sigmoid" or self.activation != "silu" or self.shared is not None or self.groups[0] > 1 \
+                or self.choice["renorm_eps"] != 1e-6:
             return None
         if self._ticket is None or self._ticket.device != residual.device:
             self._ticket = torch.zeros(1, dtype=torch.int32, device=residual.device)
@@ -163,7 +169,7 @@ class SigmoidMoE(Part):
     def forward(self, ctx, x):
         routed = self._experts(ctx, x, *kernels.moe_route_sort(
             x, self.router, self.bias, self.top_k, self.norm_topk_prob, self.routed_scaling_factor, self.scoring,
-            self.groups, self.identity))
+            self.groups, self.identity, **self.choice))
         if self.shared is None:
             return routed
         act = linear_glu(x, self.shared_w13, self.shared_interleaved, self.activation, self.shared["limit"])

@@ -1,7 +1,7 @@
 """Norms over the hidden size, fused with the residual sum that precedes them: RMSNorm
 (snowllm/ops/norm.py:11-30; snowllm/models/lfm2/layers.py:99-104) and Dynamic Tanh, which computes no
-statistics at all: tanh(alpha * x) * weight + bias with one learned number alpha; and the RMS norm in groups,
-which also reads a residual stream that is kept as several streams."""
+statistics at all: tanh(alpha * x) * weight + bias with one learned number alpha; the RMS norm in groups,
+which also reads a residual stream that is kept as several streams; and the layer norm (centred, a weight, no bias)."""
 from __future__ import annotations
 
 import torch
@@ -115,6 +115,31 @@ class GroupRMSNorm(Part):
         return self.read_streams(ctx, streams, update=update, rows=rows)
 
 
+class LayerNorm(Part):
+    """(x - mean) / sqrt(mean((x - mean)^2) + eps) * weight * gain, statistics and weight in float.  ``gain``: a constant
+    on the output (a model that scales its logits puts the factor into the norm before its head)."""
+    libraries = ("layer_norm",)
+    fusable_rms = False
+
+    def __init__(self, dtype, names, *, size: int, eps: float, gain: float = 1.0):
+        super().__init__(dtype, names)
+        self.size, self.eps, self.gain = size, float(eps), float(gain)
+        self.weight = None
+
+    def declare(self, has):
+        return [TensorSpec("weight", self.names["weight"], (self.size,), INIT_ONES, KEEP_F32)]
+
+    def bind(self, tensors):
+        self.weight = tensors["weight"]
+
+    def forward(self, ctx, residual, delta=None, rows=None):
+        """``residual += delta`` in float (a tensor, any of the deltas in pieces, or a ``kernels.NormedDelta`` with a norm
+        of its own), then the norm of the sum in the compute dtype.  With ``rows`` only those rows come out and the
+        residual stays untouched."""
+        return kernels.layer_norm(residual, delta, self.weight, self.eps, self.dtype, gain=self.gain, rows=rows)
+
+
+register_norm("layernorm", LayerNorm)
 register_norm("rmsnorm", RMSNorm)
 register_norm("group_rmsnorm", GroupRMSNorm)
 register_norm("dyt", DynamicTanh)

@@ -100,10 +100,16 @@ class BandedRotaryPosition(RotaryPosition):
     """Rotary frequencies rescaled by bands of wavelength, as Llama 3.1 does for contexts longer than the ``original``
     one: with wavelength l = 2 pi / f, a frequency is kept where l < original / high, divided by ``factor`` where l >
     original / low, and in between goes over linearly in original / l.  ``scaling`` None: the plain table.  Worked out
-    in double precision on the host and kept in float."""
+    in double precision on the host and kept in float.  ``layout``: "halves" (element i turns with element i +
+    rot_dim/2) or "pairs" (element 2i with 2i + 1); a mixer whose kernel rotates halves lays its heads out for the second
+    when its weights are bound (``halves_order``)."""
 
-    def __init__(self, *, head_dim: int, theta: float, rot_dim: int | None = None, scaling: dict | None = None):
+    def __init__(self, *, head_dim: int, theta: float, rot_dim: int | None = None, scaling: dict | None = None,
+                 layout: str = "halves"):
         super().__init__(head_dim=head_dim, theta=theta, rot_dim=rot_dim, precise=True)
+        if layout not in ("halves", "pairs"):
+            raise ValueError(f"rotary layout {layout!r} (known: halves, pairs)")
+        self.layout = layout
         self.scaling = dict(scaling) if scaling else None
 
     def frequencies(self) -> list:
@@ -124,6 +130,13 @@ class BandedRotaryPosition(RotaryPosition):
         if self._inv_freq is None or self._inv_freq.device != torch.device(device):
             self._inv_freq = torch.tensor(self.frequencies(), dtype=torch.float64).to(torch.float32).to(device)
         return self._inv_freq, self.rot_dim
+
+
+def halves_order(head_dim: int, rot_dim: int) -> list:
+    """The order of a head's elements in which neighbours that turn together (2i, 2i + 1) stand half a rotation apart:
+    the even ones of the first ``rot_dim``, the odd ones, then the rest.  Scores do not change when q and k are both
+    reordered."""
+    return [*range(0, rot_dim, 2), *range(1, rot_dim, 2), *range(rot_dim, head_dim)]
 
 
 class NoPosition:
