@@ -1,7 +1,7 @@
 """Decode and prefill throughput of the engine at the layer sizes of the LFM2.5 models, random weights.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--config 8b-a1b|dense-1.2b|dense-2.6b]
-    python bench.py --design beledra|zafopel|toderax|kuzupel|gurolix   (another design beside the closest existing model at equal size; one JSON line)
+    python bench.py --design beledra|zafopel|toderax|kuzupel|gurolix|levovik   (another design beside the closest existing model at equal size; one JSON line)
                     [--batch B] [--context C] [--dtype bfloat16|float32] [--impl ours|reference]
 
 Prints ONE JSON line.  Without flags: LFM2.5-8B-A1B sizes, 8 requests at context 8,192.
@@ -255,6 +255,44 @@ def _lfm2_moe_alternating_like(width: int, layers: int, ff: int, vocab: int = 65
     return cfg
 
 
+def _levovik(width: int, layers: int, ff: int, vocab: int = 65536) -> dict:
+    """Levovik at sizes that resemble a real model's layers: two mixers side by side in every layer, in turns softmax
+    attention with sinks beside the gated delta rule (width / 128 heads of 128 x 128, 4 taps, ranks of 128) and softmax
+    attention whose values are its keys beside gated linear attention (width / 256 heads of 128 x 256, a rank of 16);
+    attention heads of 64, one kv head per four, rescaled frequencies; side rows of 256 a layer; the first layer dense,
+    then 4 of 32 experts of ff/8 within 2 of 4 groups."""
+    heads = width // 64
+    scaling = {"factor": 32.0, "low": 1.0, "high": 4.0, "original": 8192}
+    left = {"heads": heads, "kv_heads": max(heads // 4, 1), "dim": 64, "vdim": 64, "scale": 0.125,
+            "rot": {"dims": 64, "base": 500000.0, "scaling": scaling}}
+    delta = {"heads": width // 128, "kv_heads": width // 128, "dim": 128, "vdim": 128, "conv": 4, "decay_rank": 128,
+             "gate_rank": 128}
+    linear = {"heads": max(width // 256, 1), "dim": 128, "vdim": 256, "tau": 16.0, "decay_rank": 16}
+    moe = {"kind": "moe", "expert": {"ff": ff // 8, "limit": 7.0},
+           "router": {"experts": 32, "top": 4, "scale": 1.0, "groups": {"count": 4, "keep": 2}}}
+    out = []
+    for i in range(layers):
+        mixer = {"left": left, "right": linear if i % 2 else delta, "left_scale": 0.5, "right_scale": 0.5}
+        out.append({"type": "parallel_2" if i % 2 else "parallel", "mixer": mixer,
+                    "mlp": moe if i else {"kind": "dense", "ff": ff}})
+    return {"architecture": "Levovik", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "logit_scale": 1.0, "token_side": {"dim": 256}, "layers": json.loads(json.dumps(out))}
+
+
+def _toderax_pairs_like(width: int, layers: int, ff: int, vocab: int = 65536) -> dict:
+    """The closest existing model at equal size: Toderax with a pair in every layer, attention with equal head counts that
+    sees every key (one block of 2^20 positions) beside a retention memory of the linear attention's size, one residual
+    stream, 4 of 32 experts of ff/8 without a shared one."""
+    cfg = _toderax(width, layers, ff, vocab)
+    pair = next(l for l in cfg["layers"] if l["type"] == "parallel")
+    pair["mixer"]["left"]["mask"]["size"] = 1 << 20
+    pair["mlp"].pop("shared")
+    cfg["layers"] = json.loads(json.dumps([pair] * layers))
+    cfg["norm"]["groups"] = 1
+    cfg.pop("streams")
+    return cfg
+
+
 DESIGN_SIZES = {"w2048-l12": (2048, 12, 8192), "w1024-l6": (1024, 6, 4096)}
 # design -> (its name, its configuration at a size, the closest existing model at that size, what that is)
 DESIGNS = {"beledra": ("Beledra", _beledra, ("lfm2_dense", _lfm2_like),
@@ -270,7 +308,10 @@ DESIGNS = {"beledra": ("Beledra", _beledra, ("lfm2_dense", _lfm2_like),
            "gurolix": ("Gurolix", _gurolix, ("lfm2_moe_alternating", _lfm2_moe_alternating_like),
                        "LFM2 with routed experts at equal width and depth: attention with equal head counts and size where "
                        "the design has attention, a short convolution where it has a state-space mixer, 32 experts of "
-                       "equal width")}
+                       "equal width"),
+           "levovik": ("Levovik", _levovik, ("toderax_pairs", _toderax_pairs_like),
+                       "Toderax with a pair of mixers in every layer at equal width and depth: attention with equal head "
+                       "counts and size, a matrix memory of the linear attention's size, 4 of 32 experts of equal width")}
 
 
 def design_compare(a) -> dict:

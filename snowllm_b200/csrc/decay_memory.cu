@@ -5,7 +5,7 @@
 //
 //   S_t = diag(a_t) S_(t-1) + k_t v_t^T,      o_t = S_t^T q_t
 //
-// a_t (the decay of S's rows) and k_t come in one of three forms:
+// a_t (the decay of S's rows) and k_t come in one of two forms:
 //
 //   gated  (HGRN2):     f = low + (1 - low) * sigmoid(z + b) per head and channel, from the projection
 //                       z, a bias b and a lower bound `low`;  a_t = f, k_t = 1 - f: what the gate forgets
@@ -13,8 +13,6 @@
 //   fixed  (retention): a_t = decay[head] for every row; q and k are projections whose first rot_dim
 //                       elements per head turn with the position (split halves, angle = position *
 //                       inv_freq in float), k times k_scale after the rotation.
-//   channel (gated linear attention): a_t = sigmoid(z + b)^sharp per head and channel, z float rows of their own; q and
-//                       k are projections, q times q_scale.
 //
 // The projections arrive as float rows `proj` [M, ld] (q at q_off, k or z at k_off, both [H, dk]; v at
 // v_off [H, dv]).  Gates, decays, angles, state and sums are float whatever the model's compute dtype.
@@ -48,21 +46,13 @@
 #define DM_GROUPS 32           // column groups of S per block (a group: CPT neighbouring columns)
 #define DM_TPC 8               // threads per column
 
-enum { DM_GATED = 0, DM_FIXED = 1, DM_CHANNEL = 2 };
-
-// What the third form reads beside the projections.
-struct ChannelDecay {
-  const float* z;                                          // [M, ld], its first column that of head 0, channel 0
-  long long ld;
-  float sharp, q_scale;
-};
+enum { DM_GATED = 0, DM_FIXED = 1 };
 
 // q, k and the decay a of row r of head h of one token, from its projections `pr`.
 __device__ __forceinline__ void dm_transform(const float* __restrict__ pr, int q_off, int k_off, int h, int r, int dk,
                                              int mode, const SmallVec& gate_bias, const SmallVec& gate_low,
                                              float head_decay, const float* __restrict__ inv_freq, int rot_dim,
-                                             float k_scale, int position, const ChannelDecay& ch, size_t row, float& qv,
-                                             float& kv, float& av) {
+                                             float k_scale, int position, float& qv, float& kv, float& av) {
   const float* pq = pr + q_off + h * dk;
   const float* pk = pr + k_off + h * dk;
   if (mode == DM_GATED) {
@@ -72,12 +62,6 @@ __device__ __forceinline__ void dm_transform(const float* __restrict__ pr, int q
     const float f = low + (1.f - low) / (1.f + expf(-(pk[r] + gate_bias[h * dk + r])));
     av = f;
     kv = 1.f - f;
-  } else if (mode == DM_CHANNEL) {
-    qv = pq[r] * ch.q_scale;
-    kv = pk[r];
-    // sigmoid(z)^sharp = exp(-sharp log(1 + e^-z)), accurate at both ends
-    const float z = ch.z[row * ch.ld + h * dk + r] + gate_bias[h * dk + r];
-    av = expf(-ch.sharp * (fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z)))));
   } else {
     qv = pq[r];
     kv = pk[r];
@@ -104,8 +88,8 @@ __device__ __forceinline__ void dm_transform(const float* __restrict__ pr, int q
 __global__ void __launch_bounds__(256)
 decay_memory_prepare_kernel(const float* __restrict__ proj, long long ld, int q_off, int k_off, int mode,
                             SmallVec gate_bias, SmallVec gate_low, const float* __restrict__ inv_freq, int rot_dim,
-                            float k_scale, const int* __restrict__ positions, ChannelDecay ch, float* __restrict__ prep,
-                            int M, int H, int dk) {
+                            float k_scale, const int* __restrict__ positions, float* __restrict__ prep, int M, int H,
+                            int dk) {
   pdl_begin();
   const int HD = H * dk;
   const size_t n = (size_t)M * HD;
@@ -114,10 +98,10 @@ decay_memory_prepare_kernel(const float* __restrict__ proj, long long ld, int q_
     const int h = j / dk, r = j - h * dk;
     float qv, kv, av;
     dm_transform(proj + (size_t)m * ld, q_off, k_off, h, r, dk, mode, gate_bias, gate_low, 0.f, inv_freq, rot_dim,
-                 k_scale, rot_dim ? positions[m] : 0, ch, (size_t)m, qv, kv, av);
+                 k_scale, rot_dim ? positions[m] : 0, qv, kv, av);
     prep[i] = qv;
     prep[n + i] = kv;
-    if (mode != DM_FIXED) prep[2 * n + i] = av;
+    if (mode == DM_GATED) prep[2 * n + i] = av;
   }
 }
 
@@ -133,7 +117,7 @@ decay_memory_kernel(const float* __restrict__ proj, long long ld, int q_off, int
                     const int* __restrict__ seg_start, const int* __restrict__ seg_slot,
                     float* __restrict__ state, float* __restrict__ out, int H, int dk, int dv,
                     const int4* __restrict__ pieces, float* __restrict__ work, float* __restrict__ work_decay,
-                    const float* __restrict__ prep, int M, ChannelDecay ch) {
+                    const float* __restrict__ prep, int M) {
   pdl_begin();
   extern __shared__ __align__(16) float dm_sh[];
   constexpr int RPT = DKR / DM_TPC;                      // rows of S per thread
@@ -199,7 +183,7 @@ decay_memory_kernel(const float* __restrict__ proj, long long ld, int q_off, int
         float qv = 0.f, kv = 0.f, av = 0.f;
         if (r < dk)
           dm_transform(proj + (size_t)(t0 + t) * ld, q_off, k_off, h, r, dk, mode, gate_bias, gate_low, head_decay,
-                       inv_freq, rot_dim, k_scale, rot_dim ? positions[t0 + t] : 0, ch, (size_t)(t0 + t), qv, kv, av);
+                       inv_freq, rot_dim, k_scale, rot_dim ? positions[t0 + t] : 0, qv, kv, av);
         qs[i] = qv;
         ks[i] = kv;
         as[i] = av;
@@ -214,7 +198,7 @@ decay_memory_kernel(const float* __restrict__ proj, long long ld, int q_off, int
         reinterpret_cast<float4*>(qs)[t * p4 + r4] = src[g];
         reinterpret_cast<float4*>(ks)[t * p4 + r4] = src[n4 + g];
         reinterpret_cast<float4*>(as)[t * p4 + r4] =
-            mode != DM_FIXED ? src[2 * n4 + g] : make_float4(head_decay, head_decay, head_decay, head_decay);
+            mode == DM_GATED ? src[2 * n4 + g] : make_float4(head_decay, head_decay, head_decay, head_decay);
       }
     } else {
       const size_t n = (size_t)M * H * dk;
@@ -223,7 +207,7 @@ decay_memory_kernel(const float* __restrict__ proj, long long ld, int q_off, int
         const size_t g = ((size_t)(t0 + t) * H + h) * dk + r;
         qs[t * dkp + r] = prep[g];
         ks[t * dkp + r] = prep[n + g];
-        as[t * dkp + r] = mode != DM_FIXED ? prep[2 * n + g] : head_decay;
+        as[t * dkp + r] = mode == DM_GATED ? prep[2 * n + g] : head_decay;
       }
     }
     for (int i = threadIdx.x; i < nt * DM_COLS; i += blockDim.x) {
@@ -367,7 +351,6 @@ decay_memory_scan_kernel(const int* __restrict__ cu_pieces, const int4* __restri
 // proj: float [M, ld].  mode 0 (gated): gate_bias and gate_low over [H*dk] (float or bfloat16, one flag for
 // both).  mode 1 (fixed): decay float [H]; inv_freq float [rot_dim/2] (null or rot_dim 0: no rotation),
 // positions int32 [M].  state: float [slots, H, dk, dv].  out: float [M, H*dv].
-// mode 2 (channel): gate_bias over [H*dk]; z float [M, z_ld] (its first column that of head 0, channel 0).
 // n_pieces 0: one block walks a whole segment.  Otherwise pieces int32 [n_pieces, 4], cu_pieces int32 [B+1]
 // (first piece of each segment), work float [n_pieces, H, dk, dv], work_decay float [n_pieces, H, dk], prep
 // float [3, M, H*dk] (fixed form: 2), M the rows of proj.
@@ -377,7 +360,7 @@ SNK_API int snk_decay_memory(const float* proj, long long ld, int q_off, int k_o
                              const int* cu_seqlens, const int* seg_start, const int* seg_slot, float* state,
                              float* out, int B, int H, int dk, int dv, const int* pieces, const int* cu_pieces,
                              int n_pieces, float* work, float* work_decay, float* prep, int M,
-                             const float* z, long long z_ld, float sharp, float q_scale, cudaStream_t stream) {
+                             cudaStream_t stream) {
   if (B <= 0) return 0;
   if (H <= 0 || H > 65535 || dk <= 0 || dk > 256 || dv <= 0 || dv > 32 * 65535) return SNK_ERR_SIZE;
   if (n_pieces < 0 || (n_pieces && (!pieces || !cu_pieces || !work || !work_decay || !prep || M <= 0))) return SNK_ERR_SIZE;
@@ -388,13 +371,9 @@ SNK_API int snk_decay_memory(const float* proj, long long ld, int q_off, int k_o
     if (!decay) return SNK_ERR_SIZE;
     if (!inv_freq) rot_dim = 0;
     if (rot_dim < 0 || rot_dim > dk || (rot_dim & 1) || (rot_dim && !positions)) return SNK_ERR_SIZE;
-  } else if (mode == DM_CHANNEL) {
-    if (!gate_bias || !z || z_ld < (long long)H * dk) return SNK_ERR_SIZE;
-    rot_dim = 0;
   } else {
     return SNK_ERR_SIZE;
   }
-  const ChannelDecay ch{z, z_ld, sharp, q_scale};
   // four columns a thread where the head is wide enough to fill a block that way, else one
   const int cpt = dv > 2 * DM_GROUPS ? 4 : 1;
   const int cols = DM_GROUPS * cpt;
@@ -409,7 +388,7 @@ SNK_API int snk_decay_memory(const float* proj, long long ld, int q_off, int k_o
     snk_launch(kernel, dim3(N_, H, slices), dim3(DM_TPC * DM_GROUPS), smem, stream, proj, ld, q_off, k_off,   \
                v_off, mode, SmallVec{gate_bias, gate_f32}, SmallVec{gate_low, gate_f32}, decay, inv_freq,     \
                rot_dim, k_scale, positions, cu_seqlens, seg_start, seg_slot, state, out, H, dk, dv,           \
-               reinterpret_cast<const int4*>(pieces), work, work_decay, (const float*)prep, M, ch);           \
+               reinterpret_cast<const int4*>(pieces), work, work_decay, (const float*)prep, M);               \
   } while (0)
 #define DM_LAUNCH(DKR_, PHASE_, N_)                                                                           \
   do {                                                                                                        \
@@ -430,7 +409,7 @@ SNK_API int snk_decay_memory(const float* proj, long long ld, int q_off, int k_o
     const size_t blocks = (cells + 255) / 256;
     snk_launch(decay_memory_prepare_kernel, dim3((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16)), dim3(256), 0, stream,
                proj, ld, q_off, k_off, mode, SmallVec{gate_bias, gate_f32}, SmallVec{gate_low, gate_f32}, inv_freq,
-               rot_dim, k_scale, positions, ch, prep, M, H, dk);
+               rot_dim, k_scale, positions, prep, M, H, dk);
     SNK_LAUNCH_CHECK();
     DM_PHASE(DM_COLLECT, n_pieces);
     SNK_LAUNCH_CHECK();

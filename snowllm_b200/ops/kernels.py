@@ -115,15 +115,15 @@ _SIGNATURES = {
         "snk_mlstm": [P, LL, I, I, I, I, I, P, P, I, F, P, P, P, P, P, P, P, I, I, I, I, P],
     },
     "decay_memory": {
-        "snk_decay_memory": [P, LL, I, I, I, I, P, P, I, P, P, I, F, P, P, P, P, P, P, I, I, I, I, P, P, I, P, P, P, I, P, LL, F,
-                             F, P],
+        "snk_decay_memory": [P, LL, I, I, I, I, P, P, I, P, P, I, F, P, P, P, P, P, P, I, I, I, I, P, P, I, P, P, P, I, P],
     },
     "layer_norm": {
         "snk_layer_norm": [P, P, P, F, F, P, P, P, I, P, F, P, F, F, P, P, I, I, I, P],
         "snk_side_gate": [P, P, LL, I, P, P, I, P, I, I, I, I, P],
     },
-    "delta_memory": {
-        "snk_delta_memory": [P, LL, I, I, I, P, LL, P, P, P, LL, F, F, P, P, P, P, P, I, I, I, I, I, I, I, P],
+    "channel_memory": {
+        "snk_channel_memory": [P, LL, I, I, I, P, LL, P, P, P, LL, F, F, F, P, P, P, P, P, I, I, I, I, I, I, P, P, I, P, I, P],
+        "snk_channel_memory_work": [I, I, I, I],
     },
     "streams": {
         "snk_streams_norm": [P, P, P, P, P, P, P, I, P, P, P, P, I, I, F, P, P, I, I, I, I, I, P],
@@ -142,7 +142,7 @@ _SIGNATURES = {
         "snk_sample": [P, P, P, P, P, P, I, I, P],
     },
 }
-_RESTYPES = {"snk_paged_attention_scratch_bytes": LL, "snk_gemm_tc_scratch_bytes": LL}
+_RESTYPES = {"snk_channel_memory_work": LL, "snk_paged_attention_scratch_bytes": LL, "snk_gemm_tc_scratch_bytes": LL}
 _functions: dict[str, object] = {}
 _library_of = {fn: lib for lib, fns in _SIGNATURES.items() for fn in fns}
 
@@ -2168,15 +2168,13 @@ def mlstm(proj, q_off, k_off, v_off, i_off, f_off, bias_i, bias_f, cap, cu_seqle
 
 def decay_memory(proj, q_off, k_off, v_off, cu_seqlens, seg_start, seg_slot, state, heads, dk, dv, *,
                  gate_bias=None, gate_low=None, decay=None, inv_freq=None, rot_dim=0, k_scale=1.0, positions=None,
-                 out=None, pieces=None, z=None, z_col=0, sharp=1.0, q_scale=1.0):
+                 out=None, pieces=None):
     """S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per (segment, head) over a flat batch.  ``proj``:
     float [M, width] with q at ``q_off`` and k (or the gate's pre-activation) at ``k_off`` ([heads, dk] each)
     and v at ``v_off`` ([heads, dv]).  Gated form (``gate_bias`` and ``gate_low`` over [heads*dk]): f = low +
     (1 - low) * sigmoid(z + bias), a = f, k = 1 - f, q = silu(projection).  Fixed form (``decay`` float
     [heads]): a = decay[head] for every row; the first ``rot_dim`` elements of q and k of each head turn with
-    ``positions`` (split halves, ``inv_freq`` float [rot_dim/2]); k times ``k_scale`` afterwards.  Channel form (``z``
-    float [M, width'], heads*dk columns from ``z_col`` on, and ``gate_bias``): a = sigmoid(z + bias)^sharp, q times
-    ``q_scale``.  ``state``
+    ``positions`` (split halves, ``inv_freq`` float [rot_dim/2]); k times ``k_scale`` afterwards.  ``state``
     (float [slots, heads, dk, dv]) is read unless a segment starts at 0, and brought up to date.  Returns
     the raw head outputs, float [M, heads*dv].  ``pieces`` = (int32 [n, 4] = segment, first row, rows, flags
     with 1 for a segment's first piece and 2 for its last; int32 [B+1] = first piece of each segment): every
@@ -2190,19 +2188,9 @@ def decay_memory(proj, q_off, k_off, v_off, cu_seqlens, seg_start, seg_slot, sta
     _chk(state, "memory state", torch.float32, (state.shape[0], heads, dk, dv))
     if width < max(q_off + heads * dk, k_off + heads * dk, v_off + heads * dv):
         raise KernelError(f"memory projection of width {width} is too narrow")
-    channel = z is not None
-    gated = gate_bias is not None and not channel
+    gated = gate_bias is not None
     g32 = 0
-    z_ptr, z_ld = c_void_p(0), 0
-    if channel:
-        g32 = _small(gate_bias, "decay bias", torch.float32)
-        _chk(gate_bias, "decay bias", shape=(heads * dk,))
-        _chk(z, "decay rows", torch.float32)
-        if z.dim() != 2 or z.shape[0] != M or z.shape[1] < z_col + heads * dk:
-            raise KernelError(f"decay rows of shape {tuple(z.shape)} hold no {heads * dk} columns from {z_col} on")
-        z_ptr, z_ld = c_void_p(z.data_ptr() + 4 * z_col), z.shape[1]
-        inv_freq, rot_dim = None, 0
-    elif gated:
+    if gated:
         g32 = _small(gate_bias, "gate bias", torch.float32)
         if gate_low is None or _small(gate_low, "gate lower bound", torch.float32) != g32:
             raise KernelError("gate bias and lower bound must both be given, in one dtype")
@@ -2229,14 +2217,13 @@ def decay_memory(proj, q_off, k_off, v_off, cu_seqlens, seg_start, seg_slot, sta
         _chk(cu_pieces, "first piece of each segment", torch.int32, (B + 1,))
         work = torch.empty(n_pieces, heads, dk, dv, dtype=torch.float32, device=proj.device)
         work_decay = torch.empty(n_pieces, heads, dk, dtype=torch.float32, device=proj.device)
-        prep = torch.empty(3 if gated or channel else 2, M, heads * dk, dtype=torch.float32, device=proj.device)
-    check(fn("snk_decay_memory")(_ptr(proj), width, q_off, k_off, v_off, 2 if channel else (0 if gated else 1), _ptr(gate_bias),
+        prep = torch.empty(3 if gated else 2, M, heads * dk, dtype=torch.float32, device=proj.device)
+    check(fn("snk_decay_memory")(_ptr(proj), width, q_off, k_off, v_off, 0 if gated else 1, _ptr(gate_bias),
                                  _ptr(gate_low), g32, _ptr(decay), _ptr(inv_freq), int(rot_dim), float(k_scale),
                                  _ptr(positions), _ptr(cu_seqlens), _ptr(seg_start), _ptr(seg_slot), _ptr(state),
                                  _ptr(out), B, heads, dk, dv, _ptr(table), _ptr(cu_pieces), n_pieces, _ptr(work),
-                                 _ptr(work_decay), _ptr(prep), M, z_ptr, z_ld, float(sharp),
-                                 float(q_scale), _stream()), "decay_memory",
-          launches=4 if n_pieces else 1, work=lambda: _decay_memory_work(M, B, heads, dk, dv, n_pieces, gated or channel))
+                                 _ptr(work_decay), _ptr(prep), M, _stream()), "decay_memory",
+          launches=4 if n_pieces else 1, work=lambda: _decay_memory_work(M, B, heads, dk, dv, n_pieces, gated))
     return out
 
 
@@ -2253,15 +2240,23 @@ def _decay_memory_work(M, B, H, dk, dv, pieces, gated):
             (prep + 2 * rows_v + pieces * cells * 4 + B * cells * 4, 5 * M * cells)]
 
 
-def delta_memory(u, q_off, k_off, v_off, z, z_col, bias, rate, beta, beta_col, cu_seqlens, seg_start, seg_slot, state,
-                 kv_heads, max_len, *, unit_eps: float, q_scale: float, out=None):
-    """The gated delta rule: S <- diag(a_t) S; w = sigmoid(beta_t) (v_t - S^T k_t); S <- S + k_t w^T; o_t = S^T q_t per
-    (segment, head) over a flat batch.  ``u`` [M, width] (compute dtype) holds q and k [kv_heads, dk] at ``q_off`` and
-    ``k_off``, made unit vectors here (``unit_eps`` joins the squared length; q times ``q_scale``), and v [heads, dv] at
-    ``v_off``; a = exp(rate[h] softplus(z + bias)) with ``z`` float [M, width'], heads*dk columns from ``z_col`` on,
-    ``bias`` float [heads*dk] and ``rate`` (negative) float [heads]; ``beta`` [M, width''] (compute dtype): a logit per
-    head from ``beta_col`` on.  ``state`` float [slots, heads, dk, dv] is read unless a segment starts at 0, and brought
-    up to date.  ``max_len``: the longest segment.  Returns float [M, heads * dv]."""
+MEMORY_CHUNK = 16          # tokens of a chunk of the chunked form
+
+
+def channel_memory(u, q_off, k_off, v_off, z, z_col, bias, cu_seqlens, seg_start, seg_slot, state, kv_heads, max_len, *,
+                   rate=None, beta=None, beta_col=0, sharp: float = 1.0, q_scale: float = 1.0, unit_eps: float = 0.0,
+                   pieces=None, out=None):
+    """S <- diag(a_t) S; S <- S + k_t w^T; o_t = S^T q_t per (segment, head) over a flat batch.  ``u`` [M, width] (float
+    or bfloat16) holds q and k [kv_heads, dk] at ``q_off`` and ``k_off`` and v [heads, dv] at ``v_off``; ``z`` float [M,
+    width'] heads*dk columns from ``z_col`` on, ``bias`` float [heads*dk]; q is scaled by ``q_scale``.
+
+    Delta form (``beta`` [M, width''] in u's dtype, a logit per head from ``beta_col`` on, and ``rate`` float [heads],
+    negative): w = sigmoid(beta_t) (v_t - S^T k_t), q and k made unit vectors first (``unit_eps`` joins the squared
+    length), a = exp(rate[h] softplus(z + bias)).  Linear form: w = v_t, a = sigmoid(z + bias)^sharp.
+
+    ``state`` float [slots, heads, dk, dv] is read unless a segment starts at 0, and brought up to date.  ``max_len``: the
+    longest segment.  ``pieces`` = (int32 [n, 4] = segment, first row, up to ``MEMORY_CHUNK`` rows, flags; int32 [B+1] =
+    first piece of each segment): the chunked form.  Returns float [M, heads * dv]."""
     M, width = u.shape
     dtype = u.dtype
     _chk(u, "memory rows", (torch.float32, torch.bfloat16))
@@ -2270,12 +2265,18 @@ def delta_memory(u, q_off, k_off, v_off, z, z_col, bias, rate, beta, beta_col, c
     if width < max(q_off + kv_heads * dk, k_off + kv_heads * dk, v_off + H * dv):
         raise KernelError(f"memory rows of width {width} are too narrow")
     _chk(z, "decay rows", torch.float32)
-    _chk(beta, "write strengths", dtype)
-    for name, t, need in (("decay rows", z, z_col + H * dk), ("write strengths", beta, beta_col + H)):
+    wanted = [("decay rows", z, z_col + H * dk)]
+    delta = beta is not None
+    b_ptr, b_ld = c_void_p(0), 0
+    if delta:
+        _chk(beta, "write strengths", dtype)
+        _chk(rate, "decay rate", torch.float32, (H,))
+        wanted.append(("write strengths", beta, beta_col + H))
+        b_ptr, b_ld = c_void_p(beta.data_ptr() + beta_col * beta.element_size()), beta.shape[1]
+    for name, t, need in wanted:
         if t.dim() != 2 or t.shape[0] != M or t.shape[1] < need:
             raise KernelError(f"{name} of shape {tuple(t.shape)}, want [{M}, at least {need}]")
     _chk(bias, "decay bias", torch.float32, (H * dk,))
-    _chk(rate, "decay rate", torch.float32, (H,))
     B = seg_start.numel()
     _chk(cu_seqlens, "cu_seqlens", torch.int32, (B + 1,))
     _chk(seg_start, "seg_start", torch.int32, (B,))
@@ -2283,13 +2284,29 @@ def delta_memory(u, q_off, k_off, v_off, z, z_col, bias, rate, beta, beta_col, c
     if out is None:
         out = torch.empty(M, H * dv, dtype=torch.float32, device=u.device)
     _chk(out, "memory output", torch.float32, (M, H * dv))
-    check(fn("snk_delta_memory")(
+    table = cu_pieces = work = None
+    n_pieces = per_piece = 0
+    if pieces is not None:
+        table, cu_pieces = pieces
+        n_pieces = table.shape[0]
+        _chk(table, "memory pieces", torch.int32, (n_pieces, 4))
+        _chk(cu_pieces, "first piece of each segment", torch.int32, (B + 1,))
+        per_piece = int(fn("snk_channel_memory_work")(int(delta), H, dk, dv))
+        work = torch.empty(n_pieces * per_piece, dtype=torch.float32, device=u.device)
+    rows = (2 * kv_heads * dk + H * dv) * M * u.element_size() + M * H * (dk * 4 + (u.element_size() if delta else 0))
+    cells = M * H * dk * dv
+
+    def done():
+        if not n_pieces:
+            return rows + _nbytes(out) + 2 * B * H * dk * dv * 4, (7 if delta else 5) * cells
+        chunk_bytes = n_pieces * per_piece * 4
+        return [(rows + chunk_bytes, 0),
+                (chunk_bytes + _nbytes(out) + 2 * B * H * dk * dv * 4, (7 if delta else 5) * cells)]
+    check(fn("snk_channel_memory")(
         _ptr(u), width, int(q_off), int(k_off), int(v_off), c_void_p(z.data_ptr() + 4 * z_col), z.shape[1], _ptr(bias),
-        _ptr(rate), c_void_p(beta.data_ptr() + beta_col * beta.element_size()), beta.shape[1], float(q_scale),
-        float(unit_eps), _ptr(cu_seqlens), _ptr(seg_start), _ptr(seg_slot), _ptr(state), _ptr(out), B, H, int(kv_heads),
-        dk, dv, int(max_len), code_of(dtype), _stream()), "delta_memory",
-        work=lambda: ((2 * kv_heads * dk + H * dv) * M * u.element_size() + M * H * (dk * 4 + u.element_size())
-                      + _nbytes(out) + 2 * B * H * dk * dv * 4, 7 * M * H * dk * dv))
+        _ptr(rate), b_ptr, b_ld, float(sharp), float(q_scale), float(unit_eps), _ptr(cu_seqlens), _ptr(seg_start),
+        _ptr(seg_slot), _ptr(state), _ptr(out), B, H, int(kv_heads), dk, dv, int(max_len), _ptr(table), _ptr(cu_pieces),
+        n_pieces, _ptr(work), code_of(dtype), _stream()), "channel_memory", launches=2 if n_pieces else 1, work=done)
     return out
 
 

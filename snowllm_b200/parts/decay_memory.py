@@ -11,9 +11,6 @@
   denominator.  q = W_q x and k = W_k x turn with the position on their first ``rot_dim`` elements (split
   halves), k times head_dim^(-1/2) after the rotation.  Each head's o is divided by its root mean square
   (no weight), the heads are multiplied by silu(W_g x), then the output product.
-* ``gated_linear``: a decay per head and key channel from a low-rank product, a_t = sigmoid(z)^(1/tau) with z =
-  W_b (W_a x) + bias; q = W_q x * head_dim^(-1/2), k = W_k x.  Each head's o is divided by its root mean square and
-  weighted by ``norm`` [v_head_dim] (shared by the heads), multiplied by silu(W_g x), then the output product.
 
 One fused product leaves the projections in float; gates, decays, angles, state, sums and the per-head
 statistics are float whatever the compute dtype."""
@@ -171,65 +168,5 @@ class Retention(_DecayMemory):
         return linear(heads, self.wo, out_dtype=torch.float32)
 
 
-class LowRank:
-    """W_b W_a for two thin matrices [r, in] and [out, r], kept apart; r is padded with zeros to a multiple of 8, the
-    length the tensor-core products take.  Several pairs share the two launches: their W_a side by side, their W_b on the
-    diagonal of one matrix (the zeros between them add nothing)."""
-
-    def __init__(self, pairs, what: str):
-        for a, b in pairs:
-            if a.shape[0] != b.shape[1]:
-                raise ConfigError(f"{what}: low-rank matrices of ranks {a.shape[0]} and {b.shape[1]}")
-        self.a = pad_rows(torch.cat([a for a, _ in pairs], 0), 8)
-        n, r = sum(b.shape[0] for _, b in pairs), self.a.shape[0]
-        self.b = self.a.new_zeros(n, r)
-        row = col = 0
-        for _, b in pairs:
-            self.b[row:row + b.shape[0], col:col + b.shape[1]] = b
-            row, col = row + b.shape[0], col + b.shape[1]
-
-    def __call__(self, x):
-        """Float [M, out], the pairs' outputs side by side."""
-        return linear(linear(x, self.a), self.b, out_dtype=torch.float32)
-
-
-class GatedLinear(_DecayMemory):
-    DEFAULT_RANK = 16          # of drawn weights when the configuration names none
-
-    def __init__(self, dtype, names, *, tau: float, decay_rank: int | None = None, **kw):
-        super().__init__(dtype, names, **kw)
-        self.tau, self.decay_rank = float(tau), decay_rank
-        self.low = self.decay_bias = self.norm = None
-
-    def declare(self, has):
-        W, H, dk, dv, n = self.hidden_size, self.num_heads, self.head_dim, self.v_head_dim, self.names
-        r = self.decay_rank if self.decay_rank is not None else -1
-        return [TensorSpec("q_proj", n["q_proj"], (H * dk, W)), TensorSpec("k_proj", n["k_proj"], (H * dk, W)),
-                TensorSpec("v_proj", n["v_proj"], (H * dv, W)), TensorSpec("gate_proj", n["gate_proj"], (H * dv, W)),
-                TensorSpec("decay_a", n["decay_a"], (r, W), free_default=self.DEFAULT_RANK),
-                TensorSpec("decay_b", n["decay_b"], (H * dk, r), free_default=self.DEFAULT_RANK),
-                TensorSpec("decay_bias", n["decay_bias"], (H * dk,), INIT_BIAS, KEEP_F32),
-                TensorSpec("norm", n["norm"], (dv,), INIT_ONES, KEEP_F32),
-                TensorSpec("out_proj", n["out_proj"], (W, H * dv))]
-
-    def bind(self, tensors):
-        self.w_in = pad_rows(torch.cat([tensors[k] for k in ("q_proj", "k_proj", "v_proj", "gate_proj")], 0), 16)
-        self.low = LowRank([(tensors["decay_a"], tensors["decay_b"])], "gated linear attention")
-        self.wo, self.decay_bias = tensors["out_proj"], tensors["decay_bias"].contiguous()
-        self.norm = tensors["norm"].repeat(self.num_heads).contiguous()      # one weight for every head
-
-    def forward(self, ctx, x, cache, owns_cache=True):
-        H, dk, dv = self.num_heads, self.head_dim, self.v_head_dim
-        proj = linear(x, self.w_in, out_dtype=torch.float32)
-        raw = kernels.decay_memory(proj, 0, H * dk, 2 * H * dk, ctx.cu_seqlens, ctx.seg_start, ctx.seg_slot,
-                                   cache.tensors[0], H, dk, dv, gate_bias=self.decay_bias, z=self.low(x),
-                                   sharp=1.0 / self.tau, q_scale=dk ** -0.5, pieces=self._pieces(ctx))
-        ctx.tap("memory_raw", raw)
-        heads = kernels.head_norm_gate(raw, H, dv, self.head_norm_eps, self.dtype, weight=self.norm, gate=proj,
-                                       gate_col=2 * H * dk + H * dv, gate_act="silu")
-        return linear(heads, self.wo, out_dtype=torch.float32)
-
-
-register_mixer("gated_linear", GatedLinear)
 register_mixer("hgrn2", Hgrn2)
 register_mixer("retention", Retention)
