@@ -336,23 +336,23 @@ channel_step_kernel(const MemoryIn in, const int* __restrict__ cu_seqlens, const
 }
 
 // ---------------------------------------------------------------------------------------------
-// Chunks.  What `prepare` leaves for one (chunk, head), DKP rows (dk rounded up, zeros behind) and dvp columns (dv rounded up
-// to CC_COLS), floats:
-//   A  [DKP][MR]       delta: W and the weighted q, 16 tokens each; linear: the weighted q alone
-//   K  [16][DKP]       k_j e^(G_16 - G_j), rows in the order of cc_place
-//   E  [DKP]           e^(G_16), in the same order
-//   B  [16][16]        row i, column j <= i
-//   w0 [16][dvp]
+// Chunks.  With B the 16 x 16 matrix of B_ij (j <= i), w = w0 - W S and o = q S + B w = (q - B W) S + B w0: after one product
+// with S, [W; q - B W] S, everything of the chunk is there.  What `prepare` leaves for one (chunk, head), DKP rows (dk
+// rounded up, zeros behind) and dvp columns (dv rounded up to CC_COLS), floats:
+//   A  [MR][DKP + 4]   delta: W, then q - B W, 16 tokens each; linear: the weighted q alone
+//   K  [16][DKP]       k_j e^(G_16 - G_j)
+//   E  [DKP]           e^(G_16)
+//   V  [dvp / 16][2][16][16]   per 16 columns: w0, then B w0
 #define CC_Q 16                // tokens per chunk
 #define CC_COLS 16             // columns of S per block of `scan`
 #define CC_THREADS 256
 
 __host__ __device__ constexpr int cc_rows(bool delta) { return delta ? 2 * CC_Q : CC_Q; }
+// floats of a chunk that every block of `scan` reads, and all of them
+__host__ __device__ constexpr int cc_shared(bool delta, int dkp) { return cc_rows(delta) * (dkp + 4) + (CC_Q + 1) * dkp; }
 __host__ __device__ __forceinline__ long long cc_floats(bool delta, int dkp, int dvp) {
-  return (long long)dkp * (cc_rows(delta) + CC_Q + 1) + CC_Q * CC_Q + (long long)CC_Q * dvp;
+  return cc_shared(delta, dkp) + (long long)2 * CC_Q * dvp;
 }
-// `scan` keeps rows t, t + DKP/4, t + DKP/2, t + 3 DKP/4 of S in one thread: side by side in K and E.
-template <int DKP> __device__ __forceinline__ int cc_place(int r) { return 4 * (r % (DKP / 4)) + r / (DKP / 4); }
 __device__ __forceinline__ float cc_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -392,6 +392,33 @@ __device__ __forceinline__ float cc_transpose_sum(float (&v)[N], int lane) {
   }
   return v[0];
 }
+// x <- (I + m)^-1 x for a strictly lower triangular m
+__device__ __forceinline__ void cc_solve(const float (*__restrict__ m)[CC_Q], float (&x)[CC_Q]) {
+#pragma unroll
+  for (int i = 1; i < CC_Q; ++i)
+#pragma unroll
+    for (int j = 0; j < i; j += 4) {
+      const float4 r = *reinterpret_cast<const float4*>(&m[i][j]);
+      x[i] = fmaf(-r.x, x[j], x[i]);
+      if (j + 1 < i) x[i] = fmaf(-r.y, x[j + 1], x[i]);
+      if (j + 2 < i) x[i] = fmaf(-r.z, x[j + 2], x[i]);
+      if (j + 3 < i) x[i] = fmaf(-r.w, x[j + 3], x[i]);
+    }
+}
+// row i of m x for a lower triangular m
+__device__ __forceinline__ float cc_apply(const float (*__restrict__ m)[CC_Q], const float (&x)[CC_Q], int i) {
+  float s = 0.f;
+#pragma unroll
+  for (int j = 0; j < CC_Q; j += 4)
+    if (j <= i) {
+      const float4 r = *reinterpret_cast<const float4*>(&m[i][j]);
+      s = fmaf(r.x, x[j], s);
+      if (j + 1 <= i) s = fmaf(r.y, x[j + 1], s);
+      if (j + 2 <= i) s = fmaf(r.z, x[j + 2], s);
+      if (j + 3 <= i) s = fmaf(r.w, x[j + 3], s);
+    }
+  return s;
+}
 
 // pieces: int4 per chunk = segment, first row, rows (up to CC_Q), flags.
 template <bool DELTA, typename T, int DKP>
@@ -399,12 +426,13 @@ __global__ void __launch_bounds__(CC_THREADS, 2)
 channel_prepare_kernel(const MemoryIn in, const int4* __restrict__ pieces, float* __restrict__ work, int dvp) {
   pdl_begin();
   extern __shared__ __align__(16) float cc_sh[];
-  constexpr int VL = DKP / 32, MR = cc_rows(DELTA);
+  constexpr int VL = DKP / 32, MR = cc_rows(DELTA), AP = DKP + 4;
   float* qs = cc_sh;                                       // [16][DKP]
   float* ks = qs + CC_Q * DKP;
   float* hi = ks + CC_Q * DKP;                             // G in powers of two: hi + lo
   float* lo = hi + CC_Q * DKP;
   __shared__ __align__(16) float sys[CC_Q][CC_Q];          // beta_i A_ij, j < i
+  __shared__ __align__(16) float bm[CC_Q][CC_Q];           // B_ij, j <= i
   __shared__ float bs[CC_Q];
   const int4 piece = pieces[blockIdx.x];
   const int row0 = piece.y, nt = piece.z;
@@ -412,11 +440,20 @@ channel_prepare_kernel(const MemoryIn in, const int4* __restrict__ pieces, float
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const T* u = static_cast<const T*>(in.u);
   const float rate = DELTA ? in.rate[h] : 0.f;
-  float* mine = work + ((size_t)blockIdx.x * H + h) * cc_floats(DELTA, DKP, dvp);
-  float *wa = mine, *wk = wa + DKP * MR, *we = wk + CC_Q * DKP, *wb = we + DKP, *w0 = wb + CC_Q * CC_Q;
+  float* wa = work + ((size_t)blockIdx.x * H + h) * cc_floats(DELTA, DKP, dvp);
+  float *wk = wa + MR * AP, *we = wk + CC_Q * DKP, *wv = we + DKP;
 
-  for (int i = threadIdx.x; i < CC_Q * DKP; i += CC_THREADS) {
-    const int t = i / DKP, r = i - t * DKP;
+  auto values = [&](int c, float (&x)[CC_Q]) {             // column c of v
+#pragma unroll
+    for (int i = 0; i < CC_Q; ++i)
+      x[i] = i < nt && c < dv ? to_f<T>(u[(size_t)(row0 + i) * in.u_ld + in.v_off + h * dv + c]) : 0.f;
+  };
+  float ahead[CC_Q];                                       // a thread's first column, where that is one of v: on its way
+  values((int)threadIdx.x >= DKP ? (int)threadIdx.x - DKP : dv, ahead);
+
+#pragma unroll
+  for (int n = 0; n < CC_Q * DKP / CC_THREADS; ++n) {
+    const int i = threadIdx.x + n * CC_THREADS, t = i / DKP, r = i % DKP;
     float qv = 0.f, kv = 0.f, gv = 0.f;
     if (t < nt && r < dk) {
       const T* row = u + (size_t)(row0 + t) * in.u_ld;
@@ -459,7 +496,7 @@ channel_prepare_kernel(const MemoryIn in, const int4* __restrict__ pieces, float
       hi[t * DKP + r] = top;
       lo[t * DKP + r] = (float)(run - (double)top);
     }
-    we[cc_place<DKP>(r)] = cc_exp2(hi[(CC_Q - 1) * DKP + r]);
+    we[r] = cc_exp2(hi[(CC_Q - 1) * DKP + r]);
   }
   __syncthreads();
 
@@ -490,55 +527,51 @@ channel_prepare_kernel(const MemoryIn in, const int4* __restrict__ pieces, float
       }
     const float sum = cc_transpose_sum<MR>(acc, lane);
     const int i = lane & (CC_Q - 1);
-    if (lane < CC_Q) wb[i * CC_Q + j] = sum;               // (zero above the diagonal)
+    if (lane < CC_Q) bm[i][j] = sum;                       // (zero above the diagonal)
     else if (DELTA) sys[i][j] = i > j ? bs[i] * sum : 0.f;
   }
   __syncthreads();
 
   // the system, one column a thread: W from the weighted keys, w0 from the values
-  auto solve = [&](float (&x)[CC_Q]) {
-    if constexpr (DELTA) {
-#pragma unroll
-      for (int i = 1; i < CC_Q; ++i) {
-#pragma unroll
-        for (int j4 = 0; j4 < i; j4 += 4) {
-          const float4 m = *reinterpret_cast<const float4*>(&sys[i][j4]);
-          x[i] = fmaf(-m.x, x[j4], x[i]);                  // (entries on and above the diagonal are zero)
-          if (j4 + 1 < i) x[i] = fmaf(-m.y, x[j4 + 1], x[i]);
-          if (j4 + 2 < i) x[i] = fmaf(-m.z, x[j4 + 2], x[i]);
-          if (j4 + 3 < i) x[i] = fmaf(-m.w, x[j4 + 3], x[i]);
-        }
-      }
-    }
-  };
   for (int col = threadIdx.x; col < DKP + dvp; col += CC_THREADS) {
-    float x[CC_Q];
     if (col < DKP) {
-      float* dst = wa + (size_t)col * MR;
+      float x[CC_Q];
+#pragma unroll
+      for (int i = 0; i < CC_Q; ++i) {
+        const float k = ks[i * DKP + col], gi = hi[i * DKP + col];
+        wk[i * DKP + col] = k * cc_exp2((hi[(CC_Q - 1) * DKP + col] - gi) + (lo[(CC_Q - 1) * DKP + col] - lo[i * DKP + col]));
+        x[i] = bs[i] * k * cc_exp2(gi);
+      }
       if constexpr (DELTA) {
+        cc_solve(sys, x);
 #pragma unroll
-        for (int i = 0; i < CC_Q; ++i) x[i] = bs[i] * ks[i * DKP + col] * cc_exp2(hi[i * DKP + col]);
-        solve(x);
-#pragma unroll
-        for (int i = 0; i < CC_Q; i += 4) *reinterpret_cast<float4*>(dst + i) = make_float4(x[i], x[i + 1], x[i + 2], x[i + 3]);
-        dst += CC_Q;
+        for (int i = 0; i < CC_Q; ++i) wa[i * AP + col] = x[i];
       }
 #pragma unroll
-      for (int i = 0; i < CC_Q; ++i) x[i] = qs[i * DKP + col] * cc_exp2(hi[i * DKP + col]);
-#pragma unroll
-      for (int i = 0; i < CC_Q; i += 4) *reinterpret_cast<float4*>(dst + i) = make_float4(x[i], x[i + 1], x[i + 2], x[i + 3]);
-#pragma unroll
-      for (int i = 0; i < CC_Q; ++i)
-        wk[i * DKP + cc_place<DKP>(col)] = ks[i * DKP + col] * cc_exp2((hi[(CC_Q - 1) * DKP + col] - hi[i * DKP + col]) +
-                                                        (lo[(CC_Q - 1) * DKP + col] - lo[i * DKP + col]));
+      for (int i = 0; i < CC_Q; ++i) {
+        const float q = qs[i * DKP + col] * cc_exp2(hi[i * DKP + col]);
+        wa[(MR - CC_Q + i) * AP + col] = DELTA ? q - cc_apply(bm, x, i) : q;
+      }
     } else {
       const int c = col - DKP;
+      float* dst = wv + (size_t)(c / CC_COLS) * 2 * CC_Q * CC_COLS + c % CC_COLS;
+      float x[CC_Q];
+      if (col == threadIdx.x) {
 #pragma unroll
-      for (int i = 0; i < CC_Q; ++i)
-        x[i] = i < nt && c < dv ? bs[i] * to_f<T>(u[(size_t)(row0 + i) * in.u_ld + in.v_off + h * dv + c]) : 0.f;
-      solve(x);
+        for (int i = 0; i < CC_Q; ++i) x[i] = ahead[i];
+      } else {
+        values(c, x);
+      }
+      if constexpr (DELTA) {
 #pragma unroll
-      for (int i = 0; i < CC_Q; ++i) w0[i * dvp + c] = x[i];
+        for (int i = 0; i < CC_Q; ++i) x[i] *= bs[i];
+        cc_solve(sys, x);
+      }
+#pragma unroll
+      for (int i = 0; i < CC_Q; ++i) {
+        dst[i * CC_COLS] = x[i];
+        dst[(CC_Q + i) * CC_COLS] = cc_apply(bm, x, i);
+      }
     }
   }
 }
@@ -562,21 +595,23 @@ __device__ __forceinline__ void cc_fma2(unsigned long long& c, unsigned long lon
   asm("fma.rn.f32x2 %0, %1, %2, %0;" : "+l"(c) : "l"(a), "l"(b));
 }
 
-// One block per (segment, head, CC_COLS columns): S through the segment's chunks in order.
+// One block per (segment, head, CC_COLS columns): S through the segment's chunks in order.  S lies twice: in the registers
+// of threads 0 .. DKP-1 (four neighbouring rows, four columns each), which take it past a chunk, and transposed in shared
+// memory for the product [W; q - B W] S, whose sum over S's rows is split over the eight warps.  That product runs on
+// pairs of neighbouring rows, S's step on pairs of rows with w doubled: no operand is shuffled.
 template <bool DELTA, int DKP>
-__global__ void __launch_bounds__(CC_THREADS)
+__global__ void __launch_bounds__(CC_THREADS, DKP <= 128 ? 2 : 1)
 channel_scan_kernel(const float* __restrict__ work, const int4* __restrict__ pieces, const int* __restrict__ cu_pieces,
                     const int* __restrict__ seg_start, const int* __restrict__ seg_slot, float* __restrict__ state,
                     float* __restrict__ out, int H, int dk, int dv, int dvp) {
   pdl_begin();
   extern __shared__ __align__(16) float cc_sh[];
-  constexpr int MR = cc_rows(DELTA), TR = MR / 8;          // rows of the first product a lane holds
-  constexpr int KEEP = DKP * (MR + CC_Q + 1) + CC_Q * CC_Q;        // floats of a chunk that every block reads
-  constexpr int BUF = KEEP + CC_Q * CC_COLS;
-  constexpr int KW = DKP / 8;                              // rows of S a warp takes in the first product
-  float* Ss = cc_sh + 2 * BUF;                             // [DKP][16]
-  float* part = Ss + DKP * CC_COLS;                        // [8 warps][TR][32 lanes][4]
-  float* ws = part + 8 * TR * 128;                         // [16][16]
+  constexpr int MR = cc_rows(DELTA), TR = MR / 8, AP = DKP + 4;    // TR: rows of the product a lane holds
+  constexpr int KEEP = cc_shared(DELTA, DKP), VALS = 2 * CC_Q * CC_COLS, BUF = KEEP + VALS;
+  constexpr int KW = DKP / 8;                              // rows of S a warp takes in the product
+  float* St = cc_sh + 2 * BUF;                             // [16][AP]
+  float* part = St + CC_COLS * AP;                         // [8 warps][TR][32 lanes][4]
+  float* ws = part + 8 * TR * 128;                         // [16][16][2]
   const int b = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * CC_COLS;
   const int p0 = cu_pieces[b], p1 = cu_pieces[b + 1];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -586,31 +621,32 @@ channel_scan_kernel(const float* __restrict__ work, const int4* __restrict__ pie
     if (p < p1) {
       const float* src = work + ((size_t)p * H + h) * step;
       float* dst = cc_sh + ((p - p0) & 1) * BUF;
-      for (int i = tid; i < KEEP / 4; i += CC_THREADS) cc_cp_async16(dst + 4 * i, src + 4 * i);
-      if (tid < CC_Q * CC_COLS / 4)
-        cc_cp_async16(dst + KEEP + 4 * tid, src + KEEP + (size_t)(tid >> 2) * dvp + col0 + 4 * (tid & 3));
+#pragma unroll
+      for (int n = 0; n < (KEEP / 4 + CC_THREADS - 1) / CC_THREADS; ++n) {
+        const int i = tid + n * CC_THREADS;
+        if (i < KEEP / 4) cc_cp_async16(dst + 4 * i, src + 4 * i);
+      }
+      if (tid < VALS / 4) cc_cp_async16(dst + KEEP + 4 * tid, src + KEEP + (size_t)blockIdx.z * VALS + 4 * tid);
     }
     asm volatile("cp.async.commit_group;");
   };
   load(p0);
 
-  // S: thread t < DKP holds rows t/4 + e DKP/4, columns 4 (t % 4) ..
-  const int sr = tid >> 2, sc = 4 * (tid & 3);
+  const int sr = 4 * (tid >> 2), sc = 4 * (tid & 3);       // my rows and columns of S
   float* slot = state + ((size_t)seg_slot[b] * H + h) * dk * dv;
-  float S[4][4];
+  float S[4][4];                                           // [column][row]
   if (tid < DKP) {
     const bool fresh = seg_start[b] == 0;
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int r = sr + e * (DKP / 4);
+    for (int j = 0; j < 4; ++j) {
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
-        S[e][j] = !fresh && r < dk && col0 + sc + j < dv ? slot[(size_t)r * dv + col0 + sc + j] : 0.f;
-      *reinterpret_cast<float4*>(Ss + r * CC_COLS + sc) = make_float4(S[e][0], S[e][1], S[e][2], S[e][3]);
+      for (int e = 0; e < 4; ++e)
+        S[j][e] = !fresh && sr + e < dk && col0 + sc + j < dv ? slot[(size_t)(sr + e) * dv + col0 + sc + j] : 0.f;
+      *reinterpret_cast<float4*>(St + (sc + j) * AP + sr) = make_float4(S[j][0], S[j][1], S[j][2], S[j][3]);
     }
   }
-  // where this thread's element (i, c) of the chunk's 16 x 16 outputs lies in the partial sums
-  const int i = DELTA ? ((tid & 63) >> 4) * 4 + (tid >> 6) : ((tid & 127) >> 4) * 2 + (tid >> 7), c = tid & 15;
+  // the element (i, c) of the chunk's 16 x 16 outputs that lies at place tid of the partial sums
+  const int i = ((tid & 127) >> 4) + 8 * (tid >> 7), c = ((tid >> 2) & 3) + 4 * (tid & 3);
 
   for (int p = p0; p < p1; ++p) {
     asm volatile("cp.async.wait_group 0;");
@@ -618,105 +654,88 @@ channel_scan_kernel(const float* __restrict__ work, const int4* __restrict__ pie
     load(p + 1);
     const int4 piece = pieces[p];
     const float* buf = cc_sh + ((p - p0) & 1) * BUF;
-    const float *ka = buf + DKP * MR, *ea = ka + CC_Q * DKP, *ba = ea + DKP, *w0 = buf + KEEP;
+    const float *ka = buf + MR * AP, *ea = ka + CC_Q * DKP, *va = buf + KEEP;
     {
-      // [W; q] S over this warp's rows of S
-      unsigned long long acc[TR][2];
-#pragma unroll
-      for (int r = 0; r < TR; ++r) acc[r][0] = acc[r][1] = 0ull;
-      const float* arow = buf + warp * KW * MR + TR * (lane >> 2);
-      const float* srow = Ss + warp * KW * CC_COLS + 4 * (lane & 3);
-#pragma unroll
-      for (int k = 0; k < KW; ++k) {
-        const ulonglong2 s2 = *reinterpret_cast<const ulonglong2*>(srow + k * CC_COLS);
-        float a[TR];
-        if constexpr (TR == 4) {
-          const float4 a4 = *reinterpret_cast<const float4*>(arow + k * MR);
-          a[0] = a4.x; a[1] = a4.y; a[2] = a4.z; a[3] = a4.w;
-        } else {
-          const float2 a2 = *reinterpret_cast<const float2*>(arow + k * MR);
-          a[0] = a2.x; a[1] = a2.y;
-        }
-#pragma unroll
-        for (int r = 0; r < TR; ++r) {
-          const unsigned long long aa = cc_pair(a[r], a[r]);
-          cc_fma2(acc[r][0], aa, s2.x);
-          cc_fma2(acc[r][1], aa, s2.y);
-        }
-      }
+      unsigned long long acc[TR][4];                       // rows g + 8 r, columns ct + 4 cc: sums of even and odd rows of S
 #pragma unroll
       for (int r = 0; r < TR; ++r)
-        *reinterpret_cast<ulonglong2*>(part + ((warp * TR + r) * 32 + lane) * 4) = make_ulonglong2(acc[r][0], acc[r][1]);
-    }
-    __syncthreads();
-    float o = 0.f;
-    {
-      // this element's sums over the warps: row i of W S, row i of q S
-      const float* at = part + (DELTA ? (tid >> 6) * 128 + (tid & 63) : (tid >> 7) * 128 + (tid & 127));
-      if constexpr (DELTA) {
-        float known = 0.f;
 #pragma unroll
-        for (int w = 0; w < 8; ++w) {
-          known += at[w * TR * 128];
-          o += at[w * TR * 128 + 64];
+        for (int cc = 0; cc < 4; ++cc) acc[r][cc] = 0ull;
+      const float* arow = buf + (lane >> 2) * AP + warp * KW;
+      const float* srow = St + (lane & 3) * AP + warp * KW;
+#pragma unroll
+      for (int k = 0; k < KW; k += 4) {
+        ulonglong2 a[TR], s[4];
+#pragma unroll
+        for (int cc = 0; cc < 4; ++cc) s[cc] = *reinterpret_cast<const ulonglong2*>(srow + 4 * cc * AP + k);
+#pragma unroll
+        for (int r = 0; r < TR; ++r) a[r] = *reinterpret_cast<const ulonglong2*>(arow + 8 * r * AP + k);
+#pragma unroll
+        for (int r = 0; r < TR; ++r)
+#pragma unroll
+          for (int cc = 0; cc < 4; ++cc) {
+            cc_fma2(acc[r][cc], a[r].x, s[cc].x);
+            cc_fma2(acc[r][cc], a[r].y, s[cc].y);
+          }
+      }
+#pragma unroll
+      for (int r = 0; r < TR; ++r) {
+        float v[4];
+#pragma unroll
+        for (int cc = 0; cc < 4; ++cc) {
+          const float2 t = cc_both(acc[r][cc]);
+          v[cc] = t.x + t.y;
         }
-        ws[i * CC_COLS + c] = w0[i * CC_COLS + c] - known;
-      } else {
-#pragma unroll
-        for (int w = 0; w < 8; ++w) o += at[w * TR * 128];
-        ws[i * CC_COLS + c] = w0[i * CC_COLS + c];
+        *reinterpret_cast<float4*>(part + ((warp * TR + r) * 32 + lane) * 4) = make_float4(v[0], v[1], v[2], v[3]);
       }
     }
+    if (!DELTA) *reinterpret_cast<float2*>(ws + 2 * (i * CC_COLS + c)) = make_float2(va[i * CC_COLS + c], va[i * CC_COLS + c]);
     __syncthreads();
+    float o = va[(CC_Q + i) * CC_COLS + c];
+    if constexpr (DELTA) {
+      float w = va[i * CC_COLS + c], known = 0.f;
+#pragma unroll
+      for (int n = 0; n < 8; ++n) known += part[n * TR * 128 + tid];
+      w -= known;
+      *reinterpret_cast<float2*>(ws + 2 * (i * CC_COLS + c)) = make_float2(w, w);
+      __syncthreads();
+    }
     if (tid < DKP) {                                       // S past the chunk
       unsigned long long acc[4][2];
-      const float4 e4 = *reinterpret_cast<const float4*>(ea + 4 * sr);
-      const float ev[4] = {e4.x, e4.y, e4.z, e4.w};
+      const ulonglong2 e2 = *reinterpret_cast<const ulonglong2*>(ea + sr);
+      const float2 ex = cc_both(e2.x), ey = cc_both(e2.y);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        acc[e][0] = cc_pair(ev[e] * S[e][0], ev[e] * S[e][1]);
-        acc[e][1] = cc_pair(ev[e] * S[e][2], ev[e] * S[e][3]);
+      for (int j = 0; j < 4; ++j) {
+        acc[j][0] = cc_pair(ex.x * S[j][0], ex.y * S[j][1]);
+        acc[j][1] = cc_pair(ey.x * S[j][2], ey.y * S[j][3]);
       }
 #pragma unroll
-      for (int j = 0; j < CC_Q; ++j) {
-        const ulonglong2 w2 = *reinterpret_cast<const ulonglong2*>(ws + j * CC_COLS + sc);
-        const float4 k4 = *reinterpret_cast<const float4*>(ka + j * DKP + 4 * sr);
-        const float kv[4] = {k4.x, k4.y, k4.z, k4.w};
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const unsigned long long kk = cc_pair(kv[e], kv[e]);
-          cc_fma2(acc[e][0], kk, w2.x);
-          cc_fma2(acc[e][1], kk, w2.y);
-        }
+      for (int t = 0; t < CC_Q; ++t) {
+        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(ka + t * DKP + sr);
+        const ulonglong2 w01 = *reinterpret_cast<const ulonglong2*>(ws + 2 * (t * CC_COLS + sc));
+        const ulonglong2 w23 = *reinterpret_cast<const ulonglong2*>(ws + 2 * (t * CC_COLS + sc) + 4);
+        cc_fma2(acc[0][0], k2.x, w01.x); cc_fma2(acc[0][1], k2.y, w01.x);
+        cc_fma2(acc[1][0], k2.x, w01.y); cc_fma2(acc[1][1], k2.y, w01.y);
+        cc_fma2(acc[2][0], k2.x, w23.x); cc_fma2(acc[2][1], k2.y, w23.x);
+        cc_fma2(acc[3][0], k2.x, w23.y); cc_fma2(acc[3][1], k2.y, w23.y);
       }
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float2 a = cc_both(acc[e][0]), d = cc_both(acc[e][1]);
-        S[e][0] = a.x; S[e][1] = a.y; S[e][2] = d.x; S[e][3] = d.y;
-        *reinterpret_cast<float4*>(Ss + (sr + e * (DKP / 4)) * CC_COLS + sc) = make_float4(a.x, a.y, d.x, d.y);
+      for (int j = 0; j < 4; ++j) {
+        const float2 a = cc_both(acc[j][0]), d = cc_both(acc[j][1]);
+        S[j][0] = a.x; S[j][1] = a.y; S[j][2] = d.x; S[j][3] = d.y;
+        *reinterpret_cast<float4*>(St + (sc + j) * AP + sr) = make_float4(a.x, a.y, d.x, d.y);
       }
     }
-    {
-      const float* brow = ba + i * CC_Q;                   // (zeros past the diagonal)
 #pragma unroll
-      for (int j = 0; j < CC_Q; j += 4) {
-        const float4 b4 = *reinterpret_cast<const float4*>(brow + j);
-        o = fmaf(b4.x, ws[j * CC_COLS + c], o);
-        o = fmaf(b4.y, ws[(j + 1) * CC_COLS + c], o);
-        o = fmaf(b4.z, ws[(j + 2) * CC_COLS + c], o);
-        o = fmaf(b4.w, ws[(j + 3) * CC_COLS + c], o);
-      }
-      if (i < piece.z && col0 + c < dv) out[((size_t)(piece.y + i) * H + h) * dv + col0 + c] = o;
-    }
+    for (int n = 0; n < 8; ++n) o += part[n * TR * 128 + (DELTA ? 256 : 0) + tid];
+    if (i < piece.z && col0 + c < dv) out[((size_t)(piece.y + i) * H + h) * dv + col0 + c] = o;
   }
   if (tid < DKP && p1 > p0)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int r = sr + e * (DKP / 4);
+    for (int j = 0; j < 4; ++j)
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
-        if (r < dk && col0 + sc + j < dv) slot[(size_t)r * dv + col0 + sc + j] = S[e][j];
-    }
+      for (int e = 0; e < 4; ++e)
+        if (sr + e < dk && col0 + sc + j < dv) slot[(size_t)(sr + e) * dv + col0 + sc + j] = S[j][e];
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -744,8 +763,8 @@ static int channel_memory(const MemoryIn& in, const int* cu_seqlens, const int* 
     snk_launch(prepare, dim3(n_pieces, H), dim3(CC_THREADS), psmem, stream, in, table, work, dvp);             \
     SNK_LAUNCH_CHECK();                                                                                        \
     auto scan = channel_scan_kernel<DELTA, DKP_>;                                                              \
-    const size_t ssmem = (size_t)(2 * (DKP_ * (cc_rows(DELTA) + CC_Q + 1) + CC_Q * CC_Q + CC_Q * CC_COLS) +    \
-                                  DKP_ * CC_COLS + cc_rows(DELTA) * 128 + CC_Q * CC_COLS) * sizeof(float);     \
+    const size_t ssmem = (size_t)(2 * (cc_shared(DELTA, DKP_) + 2 * CC_Q * CC_COLS) + CC_COLS * (DKP_ + 4) +   \
+                                  cc_rows(DELTA) * 128 + 2 * CC_Q * CC_COLS) * sizeof(float);                  \
     if (ssmem > 48 * 1024) cudaFuncSetAttribute(scan, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ssmem); \
     snk_launch(scan, dim3(B, H, slices), dim3(CC_THREADS), ssmem, stream, (const float*)work, table, cu_pieces, \
                seg_start, seg_slot, state, out, H, dk, dv, dvp);                                               \
