@@ -20,9 +20,10 @@
 //             w_i = beta_i (v_i - (k_i e^(G_i))^T S - sum_(j<i) A_ij w_j),   o_i = (q_i e^(G_i))^T S + sum_(j<=i) B_ij w_j
 //             S <- e^(G_16) S + sum_j (k_j e^(G_16 - G_j)) w_j^T
 //           Everything but the products with S can be worked out for all chunks at once: `prepare` leaves, per chunk and
-//           head, the weighted q, k, B and the solved system (w = w0 - W S); `scan` then takes S through the chunks in
-//           order, 16 columns a block.  No exponent is positive, so nothing overflows; G is summed in double and kept as
-//           two floats, so that G_i - G_j is exact to float however strong a decay lies before it.
+//           head, the weighted q, k and the solved system; `scan` then takes S through the chunks in order, 16 columns a
+//           block.  G is summed in double and kept as two floats, so that G_i - G_j is exact to float however strong a
+//           decay lies before it.  Where G stays small A and B are products of rows weighted by e^G and e^(-G); where it
+//           does not, every pair is weighted on its own, and no exponent is positive.
 #include "common.cuh"
 
 struct MemoryIn {
@@ -340,16 +341,17 @@ channel_step_kernel(const MemoryIn in, const int* __restrict__ cu_seqlens, const
 // with S, [W; q - B W] S, everything of the chunk is there.  What `prepare` leaves for one (chunk, head), DKP rows (dk
 // rounded up, zeros behind) and dvp columns (dv rounded up to CC_COLS), floats:
 //   A  [MR][DKP + 4]   delta: W, then q - B W, 16 tokens each; linear: the weighted q alone
-//   K  [16][DKP]       k_j e^(G_16 - G_j)
+//   K  [16][DKP + 4]   k_j e^(G_16 - G_j)
 //   E  [DKP]           e^(G_16)
 //   V  [dvp / 16][2][16][16]   per 16 columns: w0, then B w0
 #define CC_Q 16                // tokens per chunk
 #define CC_COLS 16             // columns of S per block of `scan`
 #define CC_THREADS 256
+#define CC_WEAK 100.f          // e^(-G) is formed while G stays above -100 powers of two
 
 __host__ __device__ constexpr int cc_rows(bool delta) { return delta ? 2 * CC_Q : CC_Q; }
 // floats of a chunk that every block of `scan` reads, and all of them
-__host__ __device__ constexpr int cc_shared(bool delta, int dkp) { return cc_rows(delta) * (dkp + 4) + (CC_Q + 1) * dkp; }
+__host__ __device__ constexpr int cc_shared(bool delta, int dkp) { return (cc_rows(delta) + CC_Q) * (dkp + 4) + dkp; }
 __host__ __device__ __forceinline__ long long cc_floats(bool delta, int dkp, int dvp) {
   return cc_shared(delta, dkp) + (long long)2 * CC_Q * dvp;
 }
@@ -434,6 +436,7 @@ channel_prepare_kernel(const MemoryIn in, const int4* __restrict__ pieces, float
   __shared__ __align__(16) float sys[CC_Q][CC_Q];          // beta_i A_ij, j < i
   __shared__ __align__(16) float bm[CC_Q][CC_Q];           // B_ij, j <= i
   __shared__ float bs[CC_Q];
+  __shared__ float end_hi[DKP], end_lo[DKP];               // G_16
   const int4 piece = pieces[blockIdx.x];
   const int row0 = piece.y, nt = piece.z;
   const int H = in.H, dk = in.dk, dv = in.dv, h = blockIdx.y, g = h / (H / in.G);
@@ -441,7 +444,7 @@ channel_prepare_kernel(const MemoryIn in, const int4* __restrict__ pieces, float
   const T* u = static_cast<const T*>(in.u);
   const float rate = DELTA ? in.rate[h] : 0.f;
   float* wa = work + ((size_t)blockIdx.x * H + h) * cc_floats(DELTA, DKP, dvp);
-  float *wk = wa + MR * AP, *we = wk + CC_Q * DKP, *wv = we + DKP;
+  float *wk = wa + MR * AP, *we = wk + CC_Q * AP, *wv = we + DKP;
 
   auto values = [&](int c, float (&x)[CC_Q]) {             // column c of v
 #pragma unroll
@@ -486,6 +489,7 @@ channel_prepare_kernel(const MemoryIn in, const int4* __restrict__ pieces, float
         ks[t * DKP + lane + 32 * e] *= nk;
       }
     }
+  bool strong = false;                                     // a decay that e^(-G) could not be formed for
   if (threadIdx.x < DKP) {
     const int r = threadIdx.x;
     double run = 0.0;
@@ -496,60 +500,97 @@ channel_prepare_kernel(const MemoryIn in, const int4* __restrict__ pieces, float
       hi[t * DKP + r] = top;
       lo[t * DKP + r] = (float)(run - (double)top);
     }
-    we[r] = cc_exp2(hi[(CC_Q - 1) * DKP + r]);
+    end_hi[r] = (float)run;
+    end_lo[r] = (float)(run - (double)end_hi[r]);
+    we[r] = cc_exp2(end_hi[r]);
+    strong = end_hi[r] < -CC_WEAK;
   }
-  __syncthreads();
+  strong = __syncthreads_or(strong);
+  // q e^G and k e^G in place of q and k, k e^(-G) in place of G, K
+  auto weigh = [&] {
+#pragma unroll
+    for (int n = 0; n < CC_Q * DKP / CC_THREADS; ++n) {
+      const int i = threadIdx.x + n * CC_THREADS, t = i / DKP, r = i % DKP;
+      const float top = hi[i], low = lo[i] * 0.6931471805599453f, k = ks[i];
+      const float e = cc_exp2(top);
+      const float grown = fmaf(e, low, e);
+      wk[t * AP + r] = k * cc_exp2((end_hi[r] - top) + (end_lo[r] - lo[i]));
+      qs[i] *= grown;
+      ks[i] = k * grown;
+      if (!strong) {
+        const float inv = cc_exp2(-top);
+        hi[i] = k * fmaf(inv, -low, inv);
+      }
+    }
+    __syncthreads();
+  };
+  if (!strong) weigh();
 
-  // A and B, two columns j a warp, so dealt that every warp has equal work under the triangle
+  // A and B, two columns j a warp, so dealt that every warp has equal work under the triangle: as products of weighted rows,
+  // or, where a decay within the chunk is too strong for that, pair by pair
 #pragma unroll 1
   for (int half = 0; half < 2; ++half) {
     const int j = half ? CC_Q - 1 - warp : warp;
-    float kj[VL], hj[VL], lj[VL], acc[MR];
-    cc_row<VL>(ks + j * DKP, lane, kj);
-    cc_row<VL>(hi + j * DKP, lane, hj);
-    cc_row<VL>(lo + j * DKP, lane, lj);
+    float kj[VL], acc[MR];
 #pragma unroll
     for (int i = 0; i < MR; ++i) acc[i] = 0.f;
+    if (!strong) {
+      cc_row<VL>(hi + j * DKP, lane, kj);
 #pragma unroll
-    for (int i = 0; i < CC_Q; ++i)
-      if (i >= j) {
-        float qi[VL], ki[VL], hv[VL], lv[VL];
-        cc_row<VL>(qs + i * DKP, lane, qi);
-        if (DELTA) cc_row<VL>(ks + i * DKP, lane, ki);
-        cc_row<VL>(hi + i * DKP, lane, hv);
-        cc_row<VL>(lo + i * DKP, lane, lv);
+      for (int i = 0; i < CC_Q; ++i)
+        if (i >= j) {
+          float qi[VL], ki[VL];
+          cc_row<VL>(qs + i * DKP, lane, qi);
+          if (DELTA) cc_row<VL>(ks + i * DKP, lane, ki);
 #pragma unroll
-        for (int e = 0; e < VL; ++e) {
-          const float f = kj[e] * cc_exp2((hv[e] - hj[e]) + (lv[e] - lj[e]));
-          acc[i] = fmaf(qi[e], f, acc[i]);
-          if constexpr (DELTA) acc[CC_Q + i] = fmaf(ki[e], f, acc[CC_Q + i]);
+          for (int e = 0; e < VL; ++e) {
+            acc[i] = fmaf(qi[e], kj[e], acc[i]);
+            if constexpr (DELTA) acc[CC_Q + i] = fmaf(ki[e], kj[e], acc[CC_Q + i]);
+          }
         }
-      }
+    } else {
+      float hj[VL], lj[VL];
+      cc_row<VL>(ks + j * DKP, lane, kj);
+      cc_row<VL>(hi + j * DKP, lane, hj);
+      cc_row<VL>(lo + j * DKP, lane, lj);
+#pragma unroll
+      for (int i = 0; i < CC_Q; ++i)
+        if (i >= j) {
+          float qi[VL], ki[VL], hv[VL], lv[VL];
+          cc_row<VL>(qs + i * DKP, lane, qi);
+          if (DELTA) cc_row<VL>(ks + i * DKP, lane, ki);
+          cc_row<VL>(hi + i * DKP, lane, hv);
+          cc_row<VL>(lo + i * DKP, lane, lv);
+#pragma unroll
+          for (int e = 0; e < VL; ++e) {
+            const float f = kj[e] * cc_exp2((hv[e] - hj[e]) + (lv[e] - lj[e]));
+            acc[i] = fmaf(qi[e], f, acc[i]);
+            if constexpr (DELTA) acc[CC_Q + i] = fmaf(ki[e], f, acc[CC_Q + i]);
+          }
+        }
+    }
     const float sum = cc_transpose_sum<MR>(acc, lane);
     const int i = lane & (CC_Q - 1);
     if (lane < CC_Q) bm[i][j] = sum;                       // (zero above the diagonal)
     else if (DELTA) sys[i][j] = i > j ? bs[i] * sum : 0.f;
   }
   __syncthreads();
+  if (strong) weigh();
 
   // the system, one column a thread: W from the weighted keys, w0 from the values
   for (int col = threadIdx.x; col < DKP + dvp; col += CC_THREADS) {
     if (col < DKP) {
       float x[CC_Q];
-#pragma unroll
-      for (int i = 0; i < CC_Q; ++i) {
-        const float k = ks[i * DKP + col], gi = hi[i * DKP + col];
-        wk[i * DKP + col] = k * cc_exp2((hi[(CC_Q - 1) * DKP + col] - gi) + (lo[(CC_Q - 1) * DKP + col] - lo[i * DKP + col]));
-        x[i] = bs[i] * k * cc_exp2(gi);
-      }
       if constexpr (DELTA) {
+#pragma unroll
+        for (int i = 0; i < CC_Q; ++i) x[i] = bs[i] * ks[i * DKP + col];
         cc_solve(sys, x);
 #pragma unroll
         for (int i = 0; i < CC_Q; ++i) wa[i * AP + col] = x[i];
       }
 #pragma unroll
       for (int i = 0; i < CC_Q; ++i) {
-        const float q = qs[i * DKP + col] * cc_exp2(hi[i * DKP + col]);
+        const float q = qs[i * DKP + col];
         wa[(MR - CC_Q + i) * AP + col] = DELTA ? q - cc_apply(bm, x, i) : q;
       }
     } else {
@@ -654,7 +695,7 @@ channel_scan_kernel(const float* __restrict__ work, const int4* __restrict__ pie
     load(p + 1);
     const int4 piece = pieces[p];
     const float* buf = cc_sh + ((p - p0) & 1) * BUF;
-    const float *ka = buf + MR * AP, *ea = ka + CC_Q * DKP, *va = buf + KEEP;
+    const float *ka = buf + MR * AP, *ea = ka + CC_Q * AP, *va = buf + KEEP;
     {
       unsigned long long acc[TR][4];                       // rows g + 8 r, columns ct + 4 cc: sums of even and odd rows of S
 #pragma unroll
@@ -711,7 +752,7 @@ channel_scan_kernel(const float* __restrict__ work, const int4* __restrict__ pie
       }
 #pragma unroll
       for (int t = 0; t < CC_Q; ++t) {
-        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(ka + t * DKP + sr);
+        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(ka + t * AP + sr);
         const ulonglong2 w01 = *reinterpret_cast<const ulonglong2*>(ws + 2 * (t * CC_COLS + sc));
         const ulonglong2 w23 = *reinterpret_cast<const ulonglong2*>(ws + 2 * (t * CC_COLS + sc) + 4);
         cc_fma2(acc[0][0], k2.x, w01.x); cc_fma2(acc[0][1], k2.y, w01.x);
@@ -738,6 +779,195 @@ channel_scan_kernel(const float* __restrict__ work, const int4* __restrict__ pie
         if (sr + e < dk && col0 + sc + j < dv) slot[(size_t)(sr + e) * dv + col0 + sc + j] = S[j][e];
 }
 
+// The same on the tensor cores, for bfloat16 models: S^T in the accumulators of mma.sync m16n8k16 (warp w holds 16 KS rows of S
+// by 16 columns).  Every float factor goes in as three bfloat16 terms that add up to its 24 bits, and of the nine products
+// of terms the six largest are formed: what is left out lies below float's last bit.
+__device__ __forceinline__ void cc_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// Two floats as three packed pairs of bfloat16 whose sums are the floats: each term the top half of what is left.
+__device__ __forceinline__ void cc_split3(float a, float b, uint32_t& t0, uint32_t& t1, uint32_t& t2) {
+  uint32_t ua = __float_as_uint(a), ub = __float_as_uint(b);
+  t0 = __byte_perm(ua, ub, 0x7632);
+  a -= __uint_as_float(ua & 0xffff0000u);
+  b -= __uint_as_float(ub & 0xffff0000u);
+  ua = __float_as_uint(a);
+  ub = __float_as_uint(b);
+  t1 = __byte_perm(ua, ub, 0x7632);
+  a -= __uint_as_float(ua & 0xffff0000u);
+  b -= __uint_as_float(ub & 0xffff0000u);
+  t2 = __byte_perm(__float_as_uint(a), __float_as_uint(b), 0x7632);
+}
+// c += a b over the six largest products of terms, the small ones first
+__device__ __forceinline__ void cc_mma6(float (&c)[4], const uint32_t (&a)[3][4], const uint32_t (&b0)[3], const uint32_t (&b1)[3]) {
+  cc_mma(c, a[2], b0[0], b1[0]);
+  cc_mma(c, a[1], b0[1], b1[1]);
+  cc_mma(c, a[0], b0[2], b1[2]);
+  cc_mma(c, a[1], b0[0], b1[0]);
+  cc_mma(c, a[0], b0[1], b1[1]);
+  cc_mma(c, a[0], b0[0], b1[0]);
+}
+
+#define CC_PS 20               // floats per row of the partial sums
+#define CC_WS 24               // bfloat16 per column of w's terms
+template <bool DELTA, int DKP>
+__host__ __device__ constexpr int cc_mma_warps() { return DKP / 16 < 8 ? DKP / 16 : 8; }
+
+template <bool DELTA, int DKP>
+__global__ void __launch_bounds__(CC_THREADS, DKP <= 128 ? 2 : 1)
+channel_scan_mma_kernel(const float* __restrict__ work, const int4* __restrict__ pieces, const int* __restrict__ cu_pieces,
+                        const int* __restrict__ seg_start, const int* __restrict__ seg_slot, float* __restrict__ state,
+                        float* __restrict__ out, int H, int dk, int dv, int dvp) {
+  pdl_begin();
+  extern __shared__ __align__(16) float cc_sh[];
+  constexpr int MR = cc_rows(DELTA), AP = DKP + 4;
+  constexpr int NW = cc_mma_warps<DELTA, DKP>(), KS = DKP / (16 * NW);     // warps that hold S, 16-row steps of each
+  constexpr int KEEP = cc_shared(DELTA, DKP), VALS = 2 * CC_Q * CC_COLS, BUF = KEEP + VALS;
+  float* part = cc_sh + 2 * BUF;                           // [NW][MR][CC_PS]
+  bf16* ws = reinterpret_cast<bf16*>(part + NW * MR * CC_PS);      // [3 terms][16 columns][CC_WS]
+  const int b = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * CC_COLS;
+  const int p0 = cu_pieces[b], p1 = cu_pieces[b + 1];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  const size_t step = (size_t)cc_floats(DELTA, DKP, dvp);
+
+  auto load = [&](int p) {
+    if (p < p1) {
+      const float* src = work + ((size_t)p * H + h) * step;
+      float* dst = cc_sh + ((p - p0) & 1) * BUF;
+#pragma unroll
+      for (int n = 0; n < (KEEP / 4 + CC_THREADS - 1) / CC_THREADS; ++n) {
+        const int i = tid + n * CC_THREADS;
+        if (i < KEEP / 4) cc_cp_async16(dst + 4 * i, src + 4 * i);
+      }
+      if (tid < VALS / 4) cc_cp_async16(dst + KEEP + 4 * tid, src + KEEP + (size_t)blockIdx.z * VALS + 4 * tid);
+    }
+    asm volatile("cp.async.commit_group;");
+  };
+  load(p0);
+
+  // S[k][n]: rows row0 + 16 k + 8 n + 2 t + {0, 1}, columns g (elements 0, 1) and g + 8 (2, 3)
+  float S[KS][2][4];
+  const int row0 = warp * 16 * KS;
+  float* slot = state + ((size_t)seg_slot[b] * H + h) * dk * dv;
+  if (warp < NW) {
+    const bool fresh = seg_start[b] == 0;
+#pragma unroll
+    for (int k = 0; k < KS; ++k)
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int r = row0 + 16 * k + 8 * n + 2 * t + (e & 1), c = col0 + g + 8 * (e >> 1);
+          S[k][n][e] = !fresh && r < dk && c < dv ? slot[(size_t)r * dv + c] : 0.f;
+        }
+  }
+  const int i = tid >> 4, c = tid & 15;                    // my element of the chunk's 16 x 16 outputs
+
+  for (int p = p0; p < p1; ++p) {
+    asm volatile("cp.async.wait_group 0;");
+    __syncthreads();
+    load(p + 1);
+    const int4 piece = pieces[p];
+    const float* buf = cc_sh + ((p - p0) & 1) * BUF;
+    const float *ka = buf + MR * AP, *ea = ka + CC_Q * AP, *va = buf + KEEP;
+    uint32_t kb[KS][2][2][3];                              // K's terms: tokens 2 t, 2 t + 1 (and + 8), row g of each tile
+    if (warp < NW) {
+      float acc[MR / 8][4];                                // columns g, g + 8; rows 2 t, 2 t + 1 of the product
+#pragma unroll
+      for (int m = 0; m < MR / 8; ++m)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[m][e] = 0.f;
+#pragma unroll
+      for (int k = 0; k < KS; ++k) {
+        uint32_t sa[3][4];
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          cc_split3(S[k][n][0], S[k][n][1], sa[0][2 * n], sa[1][2 * n], sa[2][2 * n]);
+          cc_split3(S[k][n][2], S[k][n][3], sa[0][2 * n + 1], sa[1][2 * n + 1], sa[2][2 * n + 1]);
+        }
+        const float* arow = buf + g * AP + row0 + 16 * k + 2 * t;
+#pragma unroll
+        for (int m = 0; m < MR / 8; ++m) {
+          const float2 lo = *reinterpret_cast<const float2*>(arow + 8 * m * AP);
+          const float2 hi = *reinterpret_cast<const float2*>(arow + 8 * m * AP + 8);
+          uint32_t b0[3], b1[3];
+          cc_split3(lo.x, lo.y, b0[0], b0[1], b0[2]);
+          cc_split3(hi.x, hi.y, b1[0], b1[1], b1[2]);
+          cc_mma6(acc[m], sa, b0, b1);
+        }
+      }
+      float* at = part + (warp * MR + 2 * t) * CC_PS + g;
+#pragma unroll
+      for (int m = 0; m < MR / 8; ++m) {
+        at[8 * m * CC_PS] = acc[m][0];
+        at[(8 * m + 1) * CC_PS] = acc[m][1];
+        at[8 * m * CC_PS + 8] = acc[m][2];
+        at[(8 * m + 1) * CC_PS + 8] = acc[m][3];
+      }
+#pragma unroll
+      for (int k = 0; k < KS; ++k)
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int q = 0; q < 2; ++q) {
+            const float* kr = ka + (2 * t + 8 * q) * AP + row0 + 16 * k + 8 * n + g;
+            cc_split3(kr[0], kr[AP], kb[k][n][q][0], kb[k][n][q][1], kb[k][n][q][2]);
+          }
+    }
+    __syncthreads();
+    float o = va[(CC_Q + i) * CC_COLS + c], w = va[i * CC_COLS + c];
+    if constexpr (DELTA) {
+      float known = 0.f;
+#pragma unroll
+      for (int n = 0; n < NW; ++n) known += part[(n * MR + i) * CC_PS + c];
+      w -= known;
+    }
+    {
+      uint32_t t0, t1, t2;
+      cc_split3(w, 0.f, t0, t1, t2);
+      unsigned short* at = reinterpret_cast<unsigned short*>(ws) + c * CC_WS + i;
+      at[0] = (unsigned short)t0;
+      at[16 * CC_WS] = (unsigned short)t1;
+      at[32 * CC_WS] = (unsigned short)t2;
+    }
+    __syncthreads();
+    if (warp < NW) {                                       // S past the chunk
+      uint32_t wa[3][4];
+#pragma unroll
+      for (int q = 0; q < 3; ++q) {
+        const bf16* at = ws + (q * 16 + g) * CC_WS + 2 * t;
+        wa[q][0] = *reinterpret_cast<const uint32_t*>(at);
+        wa[q][1] = *reinterpret_cast<const uint32_t*>(at + 8 * CC_WS);
+        wa[q][2] = *reinterpret_cast<const uint32_t*>(at + 8);
+        wa[q][3] = *reinterpret_cast<const uint32_t*>(at + 8 * CC_WS + 8);
+      }
+#pragma unroll
+      for (int k = 0; k < KS; ++k)
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          const float2 e2 = *reinterpret_cast<const float2*>(ea + row0 + 16 * k + 8 * n + 2 * t);
+          S[k][n][0] *= e2.x; S[k][n][1] *= e2.y; S[k][n][2] *= e2.x; S[k][n][3] *= e2.y;
+          cc_mma6(S[k][n], wa, kb[k][n][0], kb[k][n][1]);
+        }
+    }
+#pragma unroll
+    for (int n = 0; n < NW; ++n) o += part[(n * MR + MR - CC_Q + i) * CC_PS + c];
+    if (i < piece.z && col0 + c < dv) out[((size_t)(piece.y + i) * H + h) * dv + col0 + c] = o;
+  }
+  if (warp < NW && p1 > p0)
+#pragma unroll
+    for (int k = 0; k < KS; ++k)
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int r = row0 + 16 * k + 8 * n + 2 * t + (e & 1), cc = col0 + g + 8 * (e >> 1);
+          if (r < dk && cc < dv) slot[(size_t)r * dv + cc] = S[k][n][e];
+        }
+}
+
 // ---------------------------------------------------------------------------------------------
 static int cm_rows_padded(int dk) { return dk <= 32 ? 32 : (dk <= 64 ? 64 : (dk <= 128 ? 128 : 256)); }
 
@@ -762,9 +992,11 @@ static int channel_memory(const MemoryIn& in, const int* cu_seqlens, const int* 
     if (psmem > 48 * 1024) cudaFuncSetAttribute(prepare, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)psmem); \
     snk_launch(prepare, dim3(n_pieces, H), dim3(CC_THREADS), psmem, stream, in, table, work, dvp);             \
     SNK_LAUNCH_CHECK();                                                                                        \
-    auto scan = channel_scan_kernel<DELTA, DKP_>;                                                              \
-    const size_t ssmem = (size_t)(2 * (cc_shared(DELTA, DKP_) + 2 * CC_Q * CC_COLS) + CC_COLS * (DKP_ + 4) +   \
-                                  cc_rows(DELTA) * 128 + 2 * CC_Q * CC_COLS) * sizeof(float);                  \
+    const bool mma = dtype == SNK_BF16;                                                                        \
+    auto scan = mma ? channel_scan_mma_kernel<DELTA, DKP_> : channel_scan_kernel<DELTA, DKP_>;                 \
+    size_t ssmem = (size_t)2 * (cc_shared(DELTA, DKP_) + 2 * CC_Q * CC_COLS) * sizeof(float);                  \
+    if (mma) ssmem += (size_t)cc_mma_warps<DELTA, DKP_>() * cc_rows(DELTA) * CC_PS * sizeof(float) + 48 * CC_WS * sizeof(bf16); \
+    else ssmem += (size_t)(CC_COLS * (DKP_ + 4) + cc_rows(DELTA) * 128 + 2 * CC_Q * CC_COLS) * sizeof(float);  \
     if (ssmem > 48 * 1024) cudaFuncSetAttribute(scan, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ssmem); \
     snk_launch(scan, dim3(B, H, slices), dim3(CC_THREADS), ssmem, stream, (const float*)work, table, cu_pieces, \
                seg_start, seg_slot, state, out, H, dk, dv, dvp);                                               \
