@@ -347,6 +347,9 @@ channel_step_kernel(const MemoryIn in, const int* __restrict__ cu_seqlens, const
 #define CC_Q 16                // tokens per chunk
 #define CC_COLS 16             // columns of S per block of `scan`
 #define CC_THREADS 256
+#ifndef CC_PREPARE_BLOCKS
+#define CC_PREPARE_BLOCKS 2    // of `prepare` on an SM, by its registers
+#endif
 #define CC_WEAK 100.f          // e^(-G) is formed while G stays above -100 powers of two
 
 __host__ __device__ constexpr int cc_rows(bool delta) { return delta ? 2 * CC_Q : CC_Q; }
@@ -424,7 +427,7 @@ __device__ __forceinline__ float cc_apply(const float (*__restrict__ m)[CC_Q], c
 
 // pieces: int4 per chunk = segment, first row, rows (up to CC_Q), flags.
 template <bool DELTA, typename T, int DKP>
-__global__ void __launch_bounds__(CC_THREADS, 2)
+__global__ void __launch_bounds__(CC_THREADS, CC_PREPARE_BLOCKS)
 channel_prepare_kernel(const MemoryIn in, const int4* __restrict__ pieces, float* __restrict__ work, int dvp) {
   pdl_begin();
   extern __shared__ __align__(16) float cc_sh[];
@@ -454,19 +457,28 @@ channel_prepare_kernel(const MemoryIn in, const int4* __restrict__ pieces, float
   float ahead[CC_Q];                                       // a thread's first column, where that is one of v: on its way
   values((int)threadIdx.x >= DKP ? (int)threadIdx.x - DKP : dv, ahead);
 
+  {
+    constexpr int N = CC_Q * DKP / CC_THREADS;             // elements a thread: all loads first, then the arithmetic
+    T qv[N], kv[N];
+    float zv[N];
 #pragma unroll
-  for (int n = 0; n < CC_Q * DKP / CC_THREADS; ++n) {
-    const int i = threadIdx.x + n * CC_THREADS, t = i / DKP, r = i % DKP;
-    float qv = 0.f, kv = 0.f, gv = 0.f;
-    if (t < nt && r < dk) {
-      const T* row = u + (size_t)(row0 + t) * in.u_ld;
-      qv = to_f<T>(row[in.q_off + g * dk + r]);
-      kv = to_f<T>(row[in.k_off + g * dk + r]);
-      gv = cm_log_decay<DELTA>(in.z[(size_t)(row0 + t) * in.z_ld + h * dk + r] + in.bias[h * dk + r], rate, in.sharp);
+    for (int n = 0; n < N; ++n) {
+      const int i = threadIdx.x + n * CC_THREADS, t = i / DKP, r = i % DKP;
+      const bool ok = t < nt && r < dk;
+      const size_t row = (size_t)(row0 + (ok ? t : 0));
+      const int col = ok ? r : 0;
+      qv[n] = u[row * in.u_ld + in.q_off + g * dk + col];
+      kv[n] = u[row * in.u_ld + in.k_off + g * dk + col];
+      zv[n] = in.z[row * in.z_ld + h * dk + col];
     }
-    qs[i] = DELTA ? qv : qv * in.q_scale;
-    ks[i] = kv;
-    hi[i] = gv;
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+      const int i = threadIdx.x + n * CC_THREADS, t = i / DKP, r = i % DKP;
+      const bool ok = t < nt && r < dk;
+      qs[i] = ok ? (DELTA ? to_f<T>(qv[n]) : to_f<T>(qv[n]) * in.q_scale) : 0.f;
+      ks[i] = ok ? to_f<T>(kv[n]) : 0.f;
+      hi[i] = ok ? cm_log_decay<DELTA>(zv[n] + in.bias[h * dk + r], rate, in.sharp) : 0.f;
+    }
   }
   if (threadIdx.x < CC_Q)
     bs[threadIdx.x] = !DELTA ? 1.f : threadIdx.x < nt

@@ -93,7 +93,9 @@ class Model:
     def finish_binding(self) -> None:
         if getattr(self.head, "tied", False):
             self.head.bind({"weight": self.embedding.weight})
-        for block in self.blocks:              # an arrangement may join weights of several of its parts
+        for part in self.parts():              # a part, or an arrangement, may join weights of several of its parts
+            getattr(part, "finish_binding", lambda: None)()
+        for block in self.blocks:
             getattr(block, "finish_binding", lambda: None)()
         self.bound = True
 

@@ -912,8 +912,8 @@ def short_conv(bcx, weight, state, cu_seqlens, seg_start, seg_slot, row_seg, out
 # --- matrix products -------------------------------------------------------------------
 
 def causal_conv(u, channels: int, weight, state, cu_seqlens, seg_start, seg_slot, row_seg, out=None, bias=None,
-                silu: bool = False):
-    """Depthwise causal convolution over time on the first ``channels`` columns of ``u`` [M, width]:
+                silu: bool = False, col: int = 0):
+    """Depthwise causal convolution over time on the ``channels`` columns of ``u`` [M, width] from ``col`` on:
     y[t, c] = sum_j weight[c, j] * u~[t - taps + 1 + j, c], where u~ is the request's history (``state``
     [slots, taps-1, channels], the last taps-1 rows of earlier steps; zeros for a fresh request) followed by
     this step's rows; the state is brought up to date.  ``bias`` [channels] (in the taps' dtype) is added to the sum;
@@ -922,7 +922,7 @@ def causal_conv(u, channels: int, weight, state, cu_seqlens, seg_start, seg_slot
     dtype = u.dtype
     _chk(u, "conv input", (torch.float32, torch.bfloat16))
     C, L = weight.shape
-    if C != channels or channels > width:
+    if C != channels or col < 0 or col + channels > width:
         raise KernelError(f"conv weight {tuple(weight.shape)} over {channels} of {width} columns")
     w32 = _small(weight, "conv weight", dtype)
     _chk(state, "conv state", dtype)
@@ -935,7 +935,7 @@ def causal_conv(u, channels: int, weight, state, cu_seqlens, seg_start, seg_slot
     if bias is not None:
         _chk(bias, "conv bias", weight.dtype, (C,))
     fused = M == B and L > 1
-    check(fn("snk_causal_conv")(_ptr(u), width, _ptr(weight), w32, _ptr(state), _ptr(cu_seqlens), _ptr(seg_start),
+    check(fn("snk_causal_conv")(c_void_p(u.data_ptr() + col * u.element_size()), width, _ptr(weight), w32, _ptr(state), _ptr(cu_seqlens), _ptr(seg_start),
                                 _ptr(seg_slot), _ptr(row_seg), _ptr(out), C, M, B, C, L, _ptr(bias), int(silu), code_of(dtype),
                                 _stream()),
           "causal_conv", launches=1 if fused or L == 1 else 2,

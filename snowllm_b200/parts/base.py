@@ -48,7 +48,9 @@ class Part:
     # A part whose first product reads its input as it is may take further rows into that product:
     # ``append_input_rows(weight [n, hidden]) -> first column`` after ``bind``, and ``input_rows(ctx) -> [M, width]``,
     # the product's output, after ``forward`` of a step (an output gate on the same input then costs no product of its
-    # own).  Parts that do not offer it have no such methods.
+    # own).  The other side of it is ``ride_in(host)``, after both are bound: this part's first product moves into the
+    # host's, and its forward, which must then follow the host's, takes ``host.input_rows(ctx)`` from its column on.  Parts
+    # that do not offer them have no such methods.
 
     def parts(self):
         """Parts nested in this one (a mixer made of two mixers): the model declares and binds their tensors as

@@ -62,7 +62,19 @@ class _ChannelMemory(Part):
             raise ConfigError(f"memory heads of {head_dim} rows: the kernels keep up to {MAX_HEAD_DIM}")
         self.hidden_size, self.num_heads, self.head_dim, self.v_head_dim = hidden_size, num_heads, head_dim, v_head_dim
         self.head_norm_eps, self.decay_rank = float(head_norm_eps), decay_rank
-        self.w_in = self.wo = self.low = self.norm = None
+        self.w_in = self.wo = self.low = self.norm = self._rides = None
+
+    def ride_in(self, host) -> None:
+        """Let another part's first product on the same rows form the projections (``Part``)."""
+        self._rides = (host, host.append_input_rows(self.w_in))
+        self.w_in = None
+
+    def _projected(self, ctx, x):
+        """(the projection's rows in the compute dtype, the first of their columns)."""
+        if self._rides is not None:
+            host, col = self._rides
+            return host.input_rows(ctx), col
+        return linear(x, self.w_in), 0
 
     def _low_rank(self, rank) -> tuple:
         """(rank as a tensor dimension, what a TensorSpec says about it): the checkpoint's to choose unless given."""
@@ -99,14 +111,14 @@ class GatedLinear(_ChannelMemory):
 
     def forward(self, ctx, x, cache, owns_cache=True):
         H, dk, dv = self.num_heads, self.head_dim, self.v_head_dim
-        proj = linear(x, self.w_in)
-        raw = kernels.channel_memory(proj, 0, H * dk, 2 * H * dk, self.low(x), 0, self.decay_bias, ctx.cu_seqlens,
+        proj, col = self._projected(ctx, x)
+        raw = kernels.channel_memory(proj, col, col + H * dk, col + 2 * H * dk, self.low(x), 0, self.decay_bias, ctx.cu_seqlens,
                                      ctx.seg_start, ctx.seg_slot, cache.tensors[0], H, max(ctx.host_seg_len),
                                      sharp=1.0 / self.tau, q_scale=dk ** -0.5,
                                      pieces=memory_pieces(ctx, kernels.MEMORY_CHUNK))
         ctx.tap("memory_raw", raw)
         heads = kernels.head_norm_gate(raw, H, dv, self.head_norm_eps, self.dtype, weight=self.norm, gate=proj,
-                                       gate_col=2 * H * dk + H * dv, gate_act="silu")
+                                       gate_col=col + 2 * H * dk + H * dv, gate_act="silu")
         return linear(heads, self.wo, out_dtype=torch.float32)
 
 
@@ -159,14 +171,14 @@ class DeltaRule(_ChannelMemory):
 
     def forward(self, ctx, x, cache, owns_cache=True):
         H, G, dk, dv, C = self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim, self.conv_channels
-        proj, low = linear(x, self.w_in), self.low(x)
+        (proj, col), low = self._projected(ctx, x), self.low(x)
         history = cache.tensors[1] if self.conv_taps > 1 else proj.new_empty(1, 0, C)
         u = kernels.causal_conv(proj, C, self.conv_w, history, ctx.cu_seqlens, ctx.seg_start, ctx.seg_slot, ctx.row_seg,
-                                silu=True)
+                                silu=True, col=col)
         ctx.tap("memory_in", u)
         raw = kernels.channel_memory(u, 0, G * dk, 2 * G * dk, low, 0, self.dt_bias, ctx.cu_seqlens, ctx.seg_start,
                                      ctx.seg_slot, cache.tensors[0], G, max(ctx.host_seg_len), rate=self.rate, beta=proj,
-                                     beta_col=C, q_scale=dk ** -0.5, unit_eps=self.unit_eps,
+                                     beta_col=col + C, q_scale=dk ** -0.5, unit_eps=self.unit_eps,
                                      pieces=memory_pieces(ctx, kernels.MEMORY_CHUNK))
         ctx.tap("memory_raw", raw)
         heads = kernels.head_norm_gate(raw, H, dv, self.head_norm_eps, self.dtype, weight=self.norm, gate=low,

@@ -34,6 +34,11 @@ class SideBySide(Part):
     def parts(self):
         return (self.left, self.right)
 
+    def finish_binding(self):
+        """Both read the same rows: the right mixer's first product joins the left one's, where both offer that."""
+        if hasattr(self.left, "append_input_rows") and hasattr(self.right, "ride_in"):
+            self.right.ride_in(self.left)
+
     def cache_spec(self):
         specs = tuple(s for s in self._specs if s is not None)
         return specs if len(specs) != 1 else specs[0]
