@@ -795,7 +795,7 @@ channel_scan_kernel(const float* __restrict__ work, const int4* __restrict__ pie
 // by 16 columns).  Every float factor goes in as three bfloat16 terms that add up to its 24 bits, and of the nine products
 // of terms the six largest are formed: what is left out lies below float's last bit.
 __device__ __forceinline__ void cc_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
@@ -812,14 +812,15 @@ __device__ __forceinline__ void cc_split3(float a, float b, uint32_t& t0, uint32
   b -= __uint_as_float(ub & 0xffff0000u);
   t2 = __byte_perm(__float_as_uint(a), __float_as_uint(b), 0x7632);
 }
-// c += a b over the six largest products of terms, the small ones first
-__device__ __forceinline__ void cc_mma6(float (&c)[4], const uint32_t (&a)[3][4], const uint32_t (&b0)[3], const uint32_t (&b1)[3]) {
-  cc_mma(c, a[2], b0[0], b1[0]);
-  cc_mma(c, a[1], b0[1], b1[1]);
-  cc_mma(c, a[0], b0[2], b1[2]);
-  cc_mma(c, a[1], b0[0], b1[0]);
-  cc_mma(c, a[0], b0[1], b1[1]);
-  cc_mma(c, a[0], b0[0], b1[0]);
+// c_n += a b_n over the six largest products of terms, the small ones first; the N sums take turns, so that no product waits
+// for the one before it
+template <int N>
+__device__ __forceinline__ void cc_mma6(float (*__restrict__ c)[4], const uint32_t (&a)[3][4], const uint32_t (&b)[N][2][3]) {
+  constexpr int TA[6] = {2, 1, 0, 1, 0, 0}, TB[6] = {0, 1, 2, 0, 1, 0};
+#pragma unroll
+  for (int q = 0; q < 6; ++q)
+#pragma unroll
+    for (int n = 0; n < N; ++n) cc_mma(c[n], a[TA[q]], b[n][0][TB[q]], b[n][1][TB[q]]);
 }
 
 #define CC_PS 20               // floats per row of the partial sums
@@ -900,15 +901,15 @@ channel_scan_mma_kernel(const float* __restrict__ work, const int4* __restrict__
           cc_split3(S[k][n][2], S[k][n][3], sa[0][2 * n + 1], sa[1][2 * n + 1], sa[2][2 * n + 1]);
         }
         const float* arow = buf + g * AP + row0 + 16 * k + 2 * t;
+        uint32_t ab[MR / 8][2][3];
 #pragma unroll
-        for (int m = 0; m < MR / 8; ++m) {
-          const float2 lo = *reinterpret_cast<const float2*>(arow + 8 * m * AP);
-          const float2 hi = *reinterpret_cast<const float2*>(arow + 8 * m * AP + 8);
-          uint32_t b0[3], b1[3];
-          cc_split3(lo.x, lo.y, b0[0], b0[1], b0[2]);
-          cc_split3(hi.x, hi.y, b1[0], b1[1], b1[2]);
-          cc_mma6(acc[m], sa, b0, b1);
-        }
+        for (int m = 0; m < MR / 8; ++m)
+#pragma unroll
+          for (int q = 0; q < 2; ++q) {
+            const float2 v = *reinterpret_cast<const float2*>(arow + 8 * m * AP + 8 * q);
+            cc_split3(v.x, v.y, ab[m][q][0], ab[m][q][1], ab[m][q][2]);
+          }
+        cc_mma6<MR / 8>(acc, sa, ab);
       }
       float* at = part + (warp * MR + 2 * t) * CC_PS + g;
 #pragma unroll
@@ -961,8 +962,9 @@ channel_scan_mma_kernel(const float* __restrict__ work, const int4* __restrict__
         for (int n = 0; n < 2; ++n) {
           const float2 e2 = *reinterpret_cast<const float2*>(ea + row0 + 16 * k + 8 * n + 2 * t);
           S[k][n][0] *= e2.x; S[k][n][1] *= e2.y; S[k][n][2] *= e2.x; S[k][n][3] *= e2.y;
-          cc_mma6(S[k][n], wa, kb[k][n][0], kb[k][n][1]);
         }
+#pragma unroll
+      for (int k = 0; k < KS; ++k) cc_mma6<2>(S[k], wa, kb[k]);
     }
 #pragma unroll
     for (int n = 0; n < NW; ++n) o += part[(n * MR + MR - CC_Q + i) * CC_PS + c];
