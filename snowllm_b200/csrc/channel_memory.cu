@@ -340,7 +340,7 @@ channel_step_kernel(const MemoryIn in, const int* __restrict__ cu_seqlens, const
 // Chunks.  With B the 16 x 16 matrix of B_ij (j <= i), w = w0 - W S and o = q S + B w = (q - B W) S + B w0: after one product
 // with S, [W; q - B W] S, everything of the chunk is there.  What `prepare` leaves for one (chunk, head), DKP rows (dk
 // rounded up, zeros behind) and dvp columns (dv rounded up to CC_COLS), floats:
-//   A  [MR][DKP + 4]   delta: W, then q - B W, 16 tokens each; linear: the weighted q alone
+//   A  [MR][DKP + 8]   delta: W, then q - B W, 16 tokens each; linear: the weighted q alone
 //   K  [16][DKP + 4]   k_j e^(G_16 - G_j)
 //   E  [DKP]           e^(G_16)
 //   V  [dvp / 16][2][16][16]   per 16 columns: w0, then B w0
@@ -354,7 +354,7 @@ channel_step_kernel(const MemoryIn in, const int* __restrict__ cu_seqlens, const
 
 __host__ __device__ constexpr int cc_rows(bool delta) { return delta ? 2 * CC_Q : CC_Q; }
 // floats of a chunk that every block of `scan` reads, and all of them
-__host__ __device__ constexpr int cc_shared(bool delta, int dkp) { return (cc_rows(delta) + CC_Q) * (dkp + 4) + dkp; }
+__host__ __device__ constexpr int cc_shared(bool delta, int dkp) { return cc_rows(delta) * (dkp + 8) + CC_Q * (dkp + 4) + dkp; }
 __host__ __device__ __forceinline__ long long cc_floats(bool delta, int dkp, int dvp) {
   return cc_shared(delta, dkp) + (long long)2 * CC_Q * dvp;
 }
@@ -431,7 +431,7 @@ __global__ void __launch_bounds__(CC_THREADS, CC_PREPARE_BLOCKS)
 channel_prepare_kernel(const MemoryIn in, const int4* __restrict__ pieces, float* __restrict__ work, int dvp) {
   pdl_begin();
   extern __shared__ __align__(16) float cc_sh[];
-  constexpr int VL = DKP / 32, MR = cc_rows(DELTA), AP = DKP + 4;
+  constexpr int VL = DKP / 32, MR = cc_rows(DELTA), AP = DKP + 8, KP = DKP + 4;
   float* qs = cc_sh;                                       // [16][DKP]
   float* ks = qs + CC_Q * DKP;
   float* hi = ks + CC_Q * DKP;                             // G in powers of two: hi + lo
@@ -447,7 +447,7 @@ channel_prepare_kernel(const MemoryIn in, const int4* __restrict__ pieces, float
   const T* u = static_cast<const T*>(in.u);
   const float rate = DELTA ? in.rate[h] : 0.f;
   float* wa = work + ((size_t)blockIdx.x * H + h) * cc_floats(DELTA, DKP, dvp);
-  float *wk = wa + MR * AP, *we = wk + CC_Q * AP, *wv = we + DKP;
+  float *wk = wa + MR * AP, *we = wk + CC_Q * KP, *wv = we + DKP;
 
   auto values = [&](int c, float (&x)[CC_Q]) {             // column c of v
 #pragma unroll
@@ -526,7 +526,7 @@ channel_prepare_kernel(const MemoryIn in, const int4* __restrict__ pieces, float
       const float top = hi[i], low = lo[i] * 0.6931471805599453f, k = ks[i];
       const float e = cc_exp2(top);
       const float grown = fmaf(e, low, e);
-      wk[t * AP + r] = k * cc_exp2((end_hi[r] - top) + (end_lo[r] - lo[i]));
+      wk[t * KP + r] = k * cc_exp2((end_hi[r] - top) + (end_lo[r] - lo[i]));
       qs[i] *= grown;
       ks[i] = k * grown;
       if (!strong) {
@@ -659,7 +659,7 @@ channel_scan_kernel(const float* __restrict__ work, const int4* __restrict__ pie
                     float* __restrict__ out, int H, int dk, int dv, int dvp) {
   pdl_begin();
   extern __shared__ __align__(16) float cc_sh[];
-  constexpr int MR = cc_rows(DELTA), TR = MR / 8, AP = DKP + 4;    // TR: rows of the product a lane holds
+  constexpr int MR = cc_rows(DELTA), TR = MR / 8, AP = DKP + 8, KP = DKP + 4;    // TR: rows of the product a lane holds
   constexpr int KEEP = cc_shared(DELTA, DKP), VALS = 2 * CC_Q * CC_COLS, BUF = KEEP + VALS;
   constexpr int KW = DKP / 8;                              // rows of S a warp takes in the product
   float* St = cc_sh + 2 * BUF;                             // [16][AP]
@@ -707,7 +707,7 @@ channel_scan_kernel(const float* __restrict__ work, const int4* __restrict__ pie
     load(p + 1);
     const int4 piece = pieces[p];
     const float* buf = cc_sh + ((p - p0) & 1) * BUF;
-    const float *ka = buf + MR * AP, *ea = ka + CC_Q * AP, *va = buf + KEEP;
+    const float *ka = buf + MR * AP, *ea = ka + CC_Q * KP, *va = buf + KEEP;
     {
       unsigned long long acc[TR][4];                       // rows g + 8 r, columns ct + 4 cc: sums of even and odd rows of S
 #pragma unroll
@@ -764,7 +764,7 @@ channel_scan_kernel(const float* __restrict__ work, const int4* __restrict__ pie
       }
 #pragma unroll
       for (int t = 0; t < CC_Q; ++t) {
-        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(ka + t * AP + sr);
+        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(ka + t * KP + sr);
         const ulonglong2 w01 = *reinterpret_cast<const ulonglong2*>(ws + 2 * (t * CC_COLS + sc));
         const ulonglong2 w23 = *reinterpret_cast<const ulonglong2*>(ws + 2 * (t * CC_COLS + sc) + 4);
         cc_fma2(acc[0][0], k2.x, w01.x); cc_fma2(acc[0][1], k2.y, w01.x);
@@ -835,7 +835,7 @@ channel_scan_mma_kernel(const float* __restrict__ work, const int4* __restrict__
                         float* __restrict__ out, int H, int dk, int dv, int dvp) {
   pdl_begin();
   extern __shared__ __align__(16) float cc_sh[];
-  constexpr int MR = cc_rows(DELTA), AP = DKP + 4;
+  constexpr int MR = cc_rows(DELTA), AP = DKP + 8, KP = DKP + 4;
   constexpr int NW = cc_mma_warps<DELTA, DKP>(), KS = DKP / (16 * NW);     // warps that hold S, 16-row steps of each
   constexpr int KEEP = cc_shared(DELTA, DKP), VALS = 2 * CC_Q * CC_COLS, BUF = KEEP + VALS;
   float* part = cc_sh + 2 * BUF;                           // [NW][MR][CC_PS]
@@ -884,7 +884,7 @@ channel_scan_mma_kernel(const float* __restrict__ work, const int4* __restrict__
     load(p + 1);
     const int4 piece = pieces[p];
     const float* buf = cc_sh + ((p - p0) & 1) * BUF;
-    const float *ka = buf + MR * AP, *ea = ka + CC_Q * AP, *va = buf + KEEP;
+    const float *ka = buf + MR * AP, *ea = ka + CC_Q * KP, *va = buf + KEEP;
     uint32_t kb[KS][2][2][3];                              // K's terms: tokens 2 t, 2 t + 1 (and + 8), row g of each tile
     if (warp < NW) {
       float acc[MR / 8][4];                                // columns g, g + 8; rows 2 t, 2 t + 1 of the product
@@ -925,8 +925,8 @@ channel_scan_mma_kernel(const float* __restrict__ work, const int4* __restrict__
         for (int n = 0; n < 2; ++n)
 #pragma unroll
           for (int q = 0; q < 2; ++q) {
-            const float* kr = ka + (2 * t + 8 * q) * AP + row0 + 16 * k + 8 * n + g;
-            cc_split3(kr[0], kr[AP], kb[k][n][q][0], kb[k][n][q][1], kb[k][n][q][2]);
+            const float* kr = ka + (2 * t + 8 * q) * KP + row0 + 16 * k + 8 * n + g;
+            cc_split3(kr[0], kr[KP], kb[k][n][q][0], kb[k][n][q][1], kb[k][n][q][2]);
           }
     }
     __syncthreads();
@@ -1010,7 +1010,7 @@ static int channel_memory(const MemoryIn& in, const int* cu_seqlens, const int* 
     auto scan = mma ? channel_scan_mma_kernel<DELTA, DKP_> : channel_scan_kernel<DELTA, DKP_>;                 \
     size_t ssmem = (size_t)2 * (cc_shared(DELTA, DKP_) + 2 * CC_Q * CC_COLS) * sizeof(float);                  \
     if (mma) ssmem += (size_t)cc_mma_warps<DELTA, DKP_>() * cc_rows(DELTA) * CC_PS * sizeof(float) + 48 * CC_WS * sizeof(bf16); \
-    else ssmem += (size_t)(CC_COLS * (DKP_ + 4) + cc_rows(DELTA) * 128 + 2 * CC_Q * CC_COLS) * sizeof(float);  \
+    else ssmem += (size_t)(CC_COLS * (DKP_ + 8) + cc_rows(DELTA) * 128 + 2 * CC_Q * CC_COLS) * sizeof(float);  \
     if (ssmem > 48 * 1024) cudaFuncSetAttribute(scan, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ssmem); \
     snk_launch(scan, dim3(B, H, slices), dim3(CC_THREADS), ssmem, stream, (const float*)work, table, cu_pieces, \
                seg_start, seg_slot, state, out, H, dk, dv, dvp);                                               \
